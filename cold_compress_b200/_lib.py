@@ -134,7 +134,7 @@ def check(rc: int, what: str = "") -> int:
 
 # --------------------------------------------------------------------------- libcc_b200_seq.so (include/cc_b200_seq.h)
 SEQ_SO_PATH = Path(os.environ.get("CC_B200_SEQ_LIB", PKG / "libcc_b200_seq.so"))
-SEQ_ABI_VERSION = 4
+SEQ_ABI_VERSION = 5
 DT_F32, DT_BF16 = 0, 1
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
 
@@ -184,6 +184,7 @@ class CcSeqGatedNorm(C.Structure):
                 ("mixes", _vp), ("n_mix", _i32)]
 
 
+SCORE_SOFTMAX, SCORE_SIGMOID, SCORE_CHOSEN = range(3)
 GEMV_MAX_JOBS = 6
 
 
@@ -241,7 +242,7 @@ SEQ_EXPORTS.update({
     "cc_seq_moe_route": (C.c_int, [_vp, _i64, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
     "cc_seq_moe_group": (C.c_int, [_vp, _i32, _i32, _i32, _vp, _vp, _vp, _vp]),
     "cc_seq_gather_rows": (C.c_int, [_vp, _vp, _vp, _i32, _i32, _i32, _vp]),
-    "cc_seq_moe_expert_tokens": (C.c_int, [_vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
+    "cc_seq_moe_expert_tokens": (C.c_int, [_vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
     "cc_seq_moe_combine": (C.c_int, [C.POINTER(CcSeqMoeCombine), _vp]),
 })
 
@@ -262,7 +263,7 @@ class CcSeqSsdScan(C.Structure):
 class CcSeqDeltaScan(C.Structure):
     _fields_ = [("q", _vp), ("k", _vp), ("ldqk", _i64), ("v", _vp), ("ldv", _i64), ("beta_raw", _vp), ("ldb", _i64),
                 ("a_raw", _vp), ("lda", _i64), ("dt_bias", _vp), ("A_log", _vp), ("state", _vp), ("o", _vp)] + [
-        (n, _i32) for n in ("T", "H", "G", "D", "V")] + [("q_scale", _f32), ("unit_eps", _f32), ("qk", _vp), ("prepared", _i32)]
+        (n, _i32) for n in ("T", "H", "G", "D", "V")] + [("q_scale", _f32), ("unit_eps", _f32), ("qk", _vp), ("prepared", _i32), ("head_decay", _i32)]
 
 
 class CcSeqQkvRope(C.Structure):
@@ -303,6 +304,15 @@ SEQ_EXPORTS.update({
     "cc_seq_qk_row_norm": (C.c_int, [C.POINTER(CcSeqQkRowNorm), _vp]),
     "cc_seq_poly_norm": (C.c_int, [_vp, _i64, _vp, _vp, _i32, _i32, _i32, _f32, _vp]),
 })
+
+# ---- fifth part of the header: sublayer outputs normed before they join the stream (csrc/seq/post_kernels.cu)
+class CcSeqPostNorm(C.Structure):
+    _fields_ = [("x", _vp), ("y", _vp), ("ldy", _i64), ("wts", _vp), ("slot", _vp), ("top", _i32), ("w", _vp), ("eps", _f32),
+                ("gain_offset", _f32), ("x_out", _vp), ("x_act", _vp), ("act_dtype", _i32), ("next_w", _vp), ("next_eps", _f32),
+                ("next_offset", _f32), ("T", _i32), ("E", _i32)]
+
+
+SEQ_EXPORTS.update({"cc_seq_post_norm": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp])})
 
 _seq_lib = None
 

@@ -68,6 +68,9 @@ def _builtin():
     if "Nevodra" not in MODEL_REGISTRY:
         from .nevodra import NevodraTransformer
         register_model("Nevodra", NevodraTransformer.from_config)
+    if "Nobodra" not in MODEL_REGISTRY:
+        from .nobodra import NobodraTransformer
+        register_model("Nobodra", NobodraTransformer.from_config)
 
 
 def is_checkpoint_folder(path) -> bool:

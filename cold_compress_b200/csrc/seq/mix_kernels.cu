@@ -427,12 +427,13 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
 }
 
 // ------------------------------------------------------------------------------------------------ mixture of experts
-// A warp per token.  Scores = softmax of the router logits over all outputs; choice = score + correction; experts
-// outside the `keep` best groups (group score = its largest choice) cannot be chosen; the `top` largest choices win
-// (the lower index on a tie); weights = the winners' scores divided by their sum.
+// A warp per token.  Scores = softmax of the router logits over all outputs (or sigmoid of each); choice = score +
+// correction; experts outside the `keep` best groups (group score = its largest choice) cannot be chosen; the `top`
+// largest choices win (the lower index on a tie); weights = the winners' scores divided by their sum.  CC_SCORE_CHOSEN:
+// score = choice = logit + correction, weights = softmax over the winners (the first winner is the largest).
 __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ correction,
                                  int32_t* __restrict__ ids, float* __restrict__ wts, int T, int n, int groups, int keep, int top,
-                                 int sigmoid_scores, int group_top, int renormalize, float weight_scale) {
+                                 int scoring, int group_top, int renormalize, float weight_scale) {
     extern __shared__ float smr[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     const int t = blockIdx.x * nw + warp;
@@ -441,7 +442,9 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
     float* gm = c + n;
     if (t >= T) return;
     const float* z = logits + (size_t)t * ld;
-    if (sigmoid_scores) {
+    if (scoring == CC_SCORE_CHOSEN) {
+        for (int i = lane; i < n; i += 32) { s[i] = z[i] + (correction ? correction[i] : 0.f); c[i] = s[i]; }
+    } else if (scoring == CC_SCORE_SIGMOID) {
         for (int i = lane; i < n; i += 32) { s[i] = sigmoidf_(z[i]); c[i] = s[i] + (correction ? correction[i] : 0.f); }
     } else {
         float mx = -INFINITY;
@@ -495,7 +498,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
             if (gm[i / gs] != INFINITY) c[i] = -INFINITY;
         __syncwarp();
     }
-    float wsum = 0.f;
+    float wsum = 0.f, s0 = 0.f;
     for (int kk = 0; kk < top; ++kk) {
         float bv = -INFINITY;
         int bi = 0x7fffffff;
@@ -510,16 +513,18 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
         if (bi >= n) bi = 0;   // fewer choosable experts than `top`: a configuration error, kept harmless
+        if (kk == 0) s0 = s[bi];
+        const float sw = scoring == CC_SCORE_CHOSEN ? expf(s[bi] - s0) : s[bi];
         if (lane == 0) {
             ids[(size_t)t * top + kk] = bi;
-            wts[(size_t)t * top + kk] = s[bi];
+            wts[(size_t)t * top + kk] = sw;
             c[bi] = -INFINITY;
         }
-        wsum += s[bi];
+        wsum += sw;
         __syncwarp();
     }
     __syncwarp();
-    const float div = renormalize ? wsum + 1e-20f : 1.f;
+    const float div = scoring == CC_SCORE_CHOSEN ? wsum : (renormalize ? wsum + 1e-20f : 1.f);
     for (int kk = lane; kk < top; kk += 32) wts[(size_t)t * top + kk] = wts[(size_t)t * top + kk] / div * weight_scale;
 }
 
@@ -565,20 +570,21 @@ __global__ void gather_rows_kernel(const ST* __restrict__ src, const int32_t* __
 }
 
 // One-token form of the experts: a block of 8 warps takes 8 rows of the chosen expert's gate and up matrices for
-// one (token, choice) pair: act = silu(gate . h) * (up . h).  Pairs that chose an identity expert are skipped.
+// one (token, choice) pair: act = act(gate . h) * (up . h), or act(up . h) for experts without a gate.  Pairs that chose
+// an identity expert are skipped.
 template <typename ST>
 __global__ void __launch_bounds__(256) moe_expert_up_kernel(const ST* __restrict__ Wgu, const ST* __restrict__ h,
                                                             const int32_t* __restrict__ ids, ST* __restrict__ act,
-                                                            int n_real, int F, int E, int kind, int top) {
+                                                            int n_real, int F, int E, int kind, int top, int gated) {
     const int m = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int e = ids[m];
     const int f = blockIdx.x * 8 + warp;
     if (e >= n_real || f >= F) return;
     const int t = m / top;
     const ST* x = h + (size_t)t * E;
-    const ST* wg = Wgu + ((size_t)e * 2 * F + f) * E;
+    const ST* wg = Wgu + ((size_t)e * (gated ? 2 : 1) * F + f) * E;
     const float g = warp_dot<ST, ST>(wg, x, E, lane);
-    const float u = warp_dot<ST, ST>(wg + (size_t)F * E, x, E, lane);
+    const float u = gated ? warp_dot<ST, ST>(wg + (size_t)F * E, x, E, lane) : 1.f;
     if (lane == 0) stf(act, (size_t)m * F + f, unit_act(g, kind) * u);
 }
 
@@ -1066,15 +1072,16 @@ int cc_seq_head_norm_gate(const float* o, const float* graw, int64_t ldg, const 
 }
 
 int cc_seq_moe_route(const float* logits, int64_t ld, const float* correction, int32_t* ids, float* wts, int32_t T,
-                     int32_t n, int32_t groups, int32_t keep, int32_t top, int32_t sigmoid_scores, int32_t group_top,
+                     int32_t n, int32_t groups, int32_t keep, int32_t top, int32_t scoring, int32_t group_top,
                      int32_t renormalize, float weight_scale, void* stream) {
-    if (!logits || !ids || !wts || T < 1 || n < 1 || groups < 1 || n % groups || keep < 1 || top < 1 || top > n || group_top < 1)
+    if (!logits || !ids || !wts || T < 1 || n < 1 || groups < 1 || n % groups || keep < 1 || top < 1 || top > n || group_top < 1 ||
+        scoring < CC_SCORE_SOFTMAX || scoring > CC_SCORE_CHOSEN)
         return fail(CC_SEQ_ERR_INVALID_ARG, "moe_route: bad argument");
     const int warps = 4;
     const size_t smem = sizeof(float) * (size_t)warps * (2 * n + groups);
     if (smem > 48 * 1024) return fail(CC_SEQ_ERR_UNSUPPORTED_SHAPE, "moe_route: too many experts");
     moe_route_kernel<<<(T + warps - 1) / warps, warps * 32, smem, (cudaStream_t)stream>>>(logits, ld, correction, ids, wts, T,
-                                                                                        n, groups, keep, top, sigmoid_scores,
+                                                                                        n, groups, keep, top, scoring,
                                                                                         group_top, renormalize, weight_scale);
     return cuda_check("moe_route_kernel");
 }
@@ -1098,14 +1105,14 @@ int cc_seq_gather_rows(const void* src, const int32_t* perm, void* dst, int32_t 
 
 int cc_seq_moe_expert_tokens(const void* Wgu, const void* Wd, const void* h, const int32_t* ids, void* act, float* y,
                              int32_t dtype, int32_t T, int32_t top, int32_t n_real, int32_t F, int32_t E, int32_t kind,
-                             void* stream) {
+                             int32_t gated, void* stream) {
     if (!Wgu || !Wd || !h || !ids || !act || !y || T < 1 || top < 1 || F < 1 || E < 1 || (size_t)T * top > 65535)
         return fail(CC_SEQ_ERR_INVALID_ARG, "moe_expert_tokens: bad argument");
     cudaStream_t st = (cudaStream_t)stream;
     const dim3 gu((F + 7) / 8, T * top, 1), gd((E + 7) / 8, T * top, 1);
 #define CALL(ST)                                                                                                       \
     {                                                                                                                  \
-        moe_expert_up_kernel<ST><<<gu, 256, 0, st>>>((const ST*)Wgu, (const ST*)h, ids, (ST*)act, n_real, F, E, kind, top); \
+        moe_expert_up_kernel<ST><<<gu, 256, 0, st>>>((const ST*)Wgu, (const ST*)h, ids, (ST*)act, n_real, F, E, kind, top, gated); \
         moe_expert_down_kernel<ST><<<gd, 256, 0, st>>>((const ST*)Wd, (const ST*)act, ids, y, n_real, F, E);           \
     }
     CCM_ST(dtype, CALL);

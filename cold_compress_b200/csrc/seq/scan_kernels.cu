@@ -1,7 +1,7 @@
 // scan_kernels.cu -- sequence kernels, third part of include/cc_b200_seq.h: norms after the sum with layer scale, a
 // second (pre-normed) sublayer input and a weighted average over the depth; short causal convolutions whose tail is
-// carried from step to step; a state-space scan (scalar decay per head) and a delta-rule scan (decay per key channel),
-// both with the state of a (head, 32 value columns) tile in registers; gated group norms; rotations of query, key and
+// carried from step to step; a state-space scan (scalar decay per head) and a delta-rule scan (decay per key channel or
+// per head), both with the state of a (head, value columns) tile in registers; gated group norms; rotations of query, key and
 // value heads; the logit soft cap.
 //
 // Arithmetic rule (as in seq_kernels.cu): everything here is fp32 whatever the storage type of the neighbours; expf /
@@ -61,6 +61,10 @@ __device__ __forceinline__ float unit_act(float z, int kind) {
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) {
     const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(d), "l"(src));
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(d), "l"(src));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N>
@@ -243,7 +247,8 @@ __global__ void __launch_bounds__(512) ssd_scan_kernel(const CcSeqSsdScan a) {
 }
 
 // ------------------------------------------------------------------------------------------------ delta-rule scan
-// CTA = one head x 32 value columns.  A warp owns 4 NC columns; 8 lanes share NC columns and each keeps CH consecutive
+// CTA = one head x J value columns (32, or fewer when heads x columns / 32 would leave most of the GPU idle).  A warp owns
+// 4 NC columns; 8 lanes share NC columns and each keeps CH consecutive
 // state rows of them in registers, so the two sums over the rows that a token needs (S^T k and S^T q over the decayed state)
 // are three shuffle steps inside the warp: no shared-memory partials and no barrier per token, the warps run
 // independently through a batch.  Per batch of TB tokens (two cp.async buffers) a warp per token turns the staged rows
@@ -251,6 +256,7 @@ __global__ void __launch_bounds__(512) ssd_scan_kernel(const CcSeqSsdScan a) {
 // exp(-exp(A_log) softplus(.)) and beta.  Per token: decay the rows, the two sums, u = beta (v - S^T k), S += k u^T,
 // and o = S^T q + (q . k) u, which is the read-out of the state after the write.  The q / k / decay vectors lie in
 // shared memory in runs of CH with 4 floats of padding, so that the 8 lanes' 16-byte loads fall into different banks.
+// HD: one decay per head and token; there is no decay vector then.
 #ifndef CC_DELTA_NC
 #define CC_DELTA_NC 1
 #endif
@@ -260,9 +266,9 @@ __global__ void __launch_bounds__(512) ssd_scan_kernel(const CcSeqSsdScan a) {
 constexpr int DL_PARTS = 8, DL_NC = CC_DELTA_NC;
 
 // One token's rows turned into what the recurrence reads, by one warp: q and k as unit vectors (q times q_scale), the
-// decays, and (returned) q . k.  The same code serves the scan's own batches and the separate launch that long steps
-// use, so both give the same bits.
-template <typename LQ, typename LK, typename LA, typename SQ, typename SK, typename SG>
+// decays (per channel: lda / stg), and (returned) q . k.  The same code serves the scan's own batches and the separate
+// launch that long steps use, so both give the same bits.
+template <bool HD, typename LQ, typename LK, typename LA, typename SQ, typename SK, typename SG>
 __device__ __forceinline__ float delta_prepare_rows(int D, int lane, float q_scale, float unit_eps, float lam,
                                                     const float* __restrict__ dt_bias, LQ ldq, LK ldk, LA lda, SQ stq, SK stk, SG stg) {
     float sq = 0.f, sk = 0.f;
@@ -274,40 +280,50 @@ __device__ __forceinline__ float delta_prepare_rows(int D, int lane, float q_sca
         stq(n, qn);
         stk(n, kn);
         dot = fmaf(qn, kn, dot);
-        stg(n, expf(-lam * softplusf_(lda(n) + dt_bias[n])));
+        if constexpr (!HD) stg(n, expf(-lam * softplusf_(lda(n) + dt_bias[n])));
+    }
+    if constexpr (HD) {
+        if (lane == 0) stg(0, expf(-lam * softplusf_(lda(0) + dt_bias[0])));
     }
     return warp_sum(dot);
 }
 
 // The preparation alone, a warp per (token, head), for steps long enough that it pays to spread it over the GPU
-// instead of repeating it in every column tile of the scan: qn, kn, gd [T, H * D], beta, qk [T, H].
+// instead of repeating it in every column tile of the scan: qn, kn [T, H * D], gd [T, H * D] ([T, H]), beta, qk [T, H].
+template <bool HD>
 __global__ void delta_prepare_kernel(const CcSeqDeltaScan a, float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ gd,
                                      float* __restrict__ beta, float* __restrict__ qk) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const size_t th = (size_t)blockIdx.x * (blockDim.x >> 5) + warp;
     if (th >= (size_t)a.T * a.H) return;
     const size_t t = th / a.H;
-    const int h = (int)(th - t * a.H), g = h / (a.H / a.G), D = a.D;
+    const int h = (int)(th - t * a.H), g = h / (a.H / a.G), D = a.D, DG = HD ? 1 : D;
     const float* q = a.q + t * a.ldqk + (size_t)g * D;
     const float* k = a.k + t * a.ldqk + (size_t)g * D;
-    const float* ar = a.a_raw + t * a.lda + (size_t)h * D;
+    const float* ar = a.a_raw + t * a.lda + (size_t)h * DG;
     float* qo = qn + th * D;
     float* ko = kn + th * D;
-    float* go = gd + th * D;
-    const float dot = delta_prepare_rows(D, lane, a.q_scale, a.unit_eps, expf(a.A_log[h]), a.dt_bias + (size_t)h * D,
-                                         [&](int n) { return q[n]; }, [&](int n) { return k[n]; }, [&](int n) { return ar[n]; },
-                                         [&](int n, float v) { qo[n] = v; }, [&](int n, float v) { ko[n] = v; }, [&](int n, float v) { go[n] = v; });
+    float* go = gd + th * DG;
+    const float dot = delta_prepare_rows<HD>(D, lane, a.q_scale, a.unit_eps, expf(a.A_log[h]), a.dt_bias + (size_t)h * DG,
+                                             [&](int n) { return q[n]; }, [&](int n) { return k[n]; }, [&](int n) { return ar[n]; },
+                                             [&](int n, float v) { qo[n] = v; }, [&](int n, float v) { ko[n] = v; }, [&](int n, float v) { go[n] = v; });
     if (lane == 0) { qk[th] = dot; beta[th] = sigmoidf_(a.beta_raw[t * a.ldb + h]); }
 }
 
-template <int CH, int NC, int TB>
-__global__ void __launch_bounds__(SCAN_J / (4 * NC) * 32, 2) delta_scan_kernel(const CcSeqDeltaScan a) {
+// floats of one staging buffer: q and k (and decay) vectors, J values, beta, q . k (and the head's decay) per token
+__host__ __device__ constexpr int delta_buf_floats(int Dp, int J, int TB, bool HD) {
+    return (TB * ((HD ? 2 : 3) * Dp + J + (HD ? 3 : 2)) + 3) & ~3;
+}
+
+template <int CH, int NC, int TB, int J, bool HD>
+__global__ void __launch_bounds__(J / (4 * NC) * 32, J >= 32 ? 2 : 4) delta_scan_kernel(const CcSeqDeltaScan a) {
     extern __shared__ float4 sm_dl4[];
     float* sm = reinterpret_cast<float*>(sm_dl4);
-    constexpr int NW = SCAN_J / (4 * NC), RUN = CH + 4, Dp = DL_PARTS * RUN, NTH = NW * 32;
-    constexpr int buf_floats = TB * (3 * Dp + SCAN_J + 2);
+    constexpr int NW = J / (4 * NC), RUN = CH + 4, Dp = DL_PARTS * RUN, NTH = NW * 32;
+    constexpr int buf_floats = delta_buf_floats(Dp, J, TB, HD);
+    constexpr int O_V = (HD ? 2 : 3) * TB * Dp, O_BETA = O_V + TB * J, O_QK = O_BETA + TB, O_DEC = O_QK + TB;   // offsets in a buffer
     const int D = a.D;
-    const int h = blockIdx.x, j0 = blockIdx.y * SCAN_J, g = h / (a.H / a.G);
+    const int h = blockIdx.x, j0 = blockIdx.y * J, g = h / (a.H / a.G);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int jl = (warp * 4 + (lane >> 3)) * NC, p = lane & 7, j = j0 + jl;      // this lane's first column
     const int n0 = p * CH;
@@ -321,26 +337,40 @@ __global__ void __launch_bounds__(SCAN_J / (4 * NC) * 32, 2) delta_scan_kernel(c
     __syncthreads();
     const float lam = expf(a.A_log[h]);
     auto at = [](int n) { return (n / CH) * RUN + (n % CH); };
+    const bool vec = a.prepared && (D & 3) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.a_raw) & 15) == 0 && (a.ldqk & 3) == 0 &&
+                     (HD || (a.lda & 3) == 0);
     auto fetch = [&](int tb, float* buf) {
         const int nt = min(TB, a.T - tb);
-        // thread -> (token lane, channel): no division per copy
-        const int lanes_t = D <= NTH / 2 ? NTH / ((D + 31) / 32 * 32) : 1, width = NTH / lanes_t;
-        const int t0 = tid / width, nb = tid - t0 * width;
-        for (int t = t0; t < nt; t += lanes_t)
-            for (int n = nb; n < D; n += width) {
-                const int o = t * Dp + at(n);
+        if (vec) {      // prepared rows: 16 bytes per copy (a run of CH is a multiple of 4 floats)
+            const int d4 = D >> 2;
+            for (int idx = tid; idx < nt * d4; idx += NTH) {
+                const int t = idx / d4, n = (idx - t * d4) * 4, o = t * Dp + at(n);
                 const size_t row = (size_t)(tb + t) * a.ldqk + (size_t)g * D + n;
-                cp_async4(buf + o, a.q + row);
-                cp_async4(buf + TB * Dp + o, a.k + row);
-                cp_async4(buf + 2 * TB * Dp + o, a.a_raw + (size_t)(tb + t) * a.lda + (size_t)h * D + n);
+                cp_async16(buf + o, a.q + row);
+                cp_async16(buf + TB * Dp + o, a.k + row);
+                if constexpr (!HD) cp_async16(buf + 2 * TB * Dp + o, a.a_raw + (size_t)(tb + t) * a.lda + (size_t)h * D + n);
             }
-        for (int idx = tid; idx < nt * SCAN_J; idx += NTH) {
-            const int t = idx / SCAN_J, c = idx - t * SCAN_J;
-            if (j0 + c < a.V) cp_async4(buf + 3 * TB * Dp + idx, a.v + (size_t)(tb + t) * a.ldv + (size_t)h * a.V + j0 + c);
+        } else {
+            // thread -> (token lane, channel): no division per copy
+            const int lanes_t = D <= NTH / 2 ? NTH / ((D + 31) / 32 * 32) : 1, width = NTH / lanes_t;
+            const int t0 = tid / width, nb = tid - t0 * width;
+            for (int t = t0; t < nt; t += lanes_t)
+                for (int n = nb; n < D; n += width) {
+                    const int o = t * Dp + at(n);
+                    const size_t row = (size_t)(tb + t) * a.ldqk + (size_t)g * D + n;
+                    cp_async4(buf + o, a.q + row);
+                    cp_async4(buf + TB * Dp + o, a.k + row);
+                    if constexpr (!HD) cp_async4(buf + 2 * TB * Dp + o, a.a_raw + (size_t)(tb + t) * a.lda + (size_t)h * D + n);
+                }
         }
-        if (tid < nt) {
-            cp_async4(buf + 3 * TB * Dp + TB * SCAN_J + tid, a.beta_raw + (size_t)(tb + tid) * a.ldb + h);
-            if (a.prepared) cp_async4(buf + 3 * TB * Dp + TB * SCAN_J + TB + tid, a.qk + (size_t)(tb + tid) * a.H + h);
+        for (int idx = tid; idx < nt * J; idx += NTH) {
+            const int t = idx / J, c = idx - t * J;
+            if (j0 + c < a.V) cp_async4(buf + O_V + idx, a.v + (size_t)(tb + t) * a.ldv + (size_t)h * a.V + j0 + c);
+        }
+        for (int t = tid; t < nt; t += NTH) {
+            cp_async4(buf + O_BETA + t, a.beta_raw + (size_t)(tb + t) * a.ldb + h);
+            if (a.prepared) cp_async4(buf + O_QK + t, a.qk + (size_t)(tb + t) * a.H + h);
+            if constexpr (HD) cp_async4(buf + O_DEC + t, a.a_raw + (size_t)(tb + t) * a.lda + h);
         }
         cp_async_commit();
     };
@@ -352,34 +382,38 @@ __global__ void __launch_bounds__(SCAN_J / (4 * NC) * 32, 2) delta_scan_kernel(c
         if (tb + TB < a.T) { fetch(tb + TB, sm + (cur ^ 1) * buf_floats); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
-        float* betas = buf + 3 * TB * Dp + TB * SCAN_J;
-        float* qks = betas + TB;
+        float* betas = buf + O_BETA;
+        float* qks = buf + O_QK;
+        float* decs = buf + O_DEC;
         if (!a.prepared) {
             for (int t = warp; t < nt; t += NW) {     // a warp per token
                 float* q = buf + t * Dp;
                 float* k = buf + TB * Dp + t * Dp;
-                float* gd = buf + 2 * TB * Dp + t * Dp;
-                const float dot = delta_prepare_rows(D, lane, a.q_scale, a.unit_eps, lam, a.dt_bias + (size_t)h * D,
-                                                     [&](int n) { return q[at(n)]; }, [&](int n) { return k[at(n)]; }, [&](int n) { return gd[at(n)]; },
-                                                     [&](int n, float v) { q[at(n)] = v; }, [&](int n, float v) { k[at(n)] = v; },
-                                                     [&](int n, float v) { gd[at(n)] = v; });
+                float* gd = HD ? decs + t : buf + 2 * TB * Dp + t * Dp;
+                const float dot = delta_prepare_rows<HD>(D, lane, a.q_scale, a.unit_eps, lam, a.dt_bias + (size_t)h * (HD ? 1 : D),
+                                                         [&](int n) { return q[at(n)]; }, [&](int n) { return k[at(n)]; }, [&](int n) { return gd[at(n)]; },
+                                                         [&](int n, float v) { q[at(n)] = v; }, [&](int n, float v) { k[at(n)] = v; },
+                                                         [&](int n, float v) { gd[at(n)] = v; });
                 if (lane == 0) { qks[t] = dot; betas[t] = sigmoidf_(betas[t]); }
             }
             __syncthreads();
         }
         const float4* __restrict__ q4 = reinterpret_cast<const float4*>(buf + p * RUN);
         const float4* __restrict__ k4 = reinterpret_cast<const float4*>(buf + TB * Dp + p * RUN);
-        const float4* __restrict__ g4 = reinterpret_cast<const float4*>(buf + 2 * TB * Dp + p * RUN);
-        const float* __restrict__ vs = buf + 3 * TB * Dp;
+        const float4* __restrict__ g4 = reinterpret_cast<const float4*>(buf + 2 * TB * Dp + p * RUN);   // per-channel decays only
+        const float* __restrict__ vs = buf + O_V;
         float* orow = a.o + (size_t)tb * a.H * a.V + (size_t)h * a.V + j;
 #pragma unroll 2
         for (int t = 0; t < nt; ++t) {
             float kk[CH], rk[NC], rq[NC];
 #pragma unroll
             for (int e = 0; e < NC; ++e) rk[e] = rq[e] = 0.f;
+            const float dec = HD ? decs[t] : 1.f;
 #pragma unroll
             for (int c4 = 0; c4 < CH / 4; ++c4) {
-                const float4 gv = g4[t * (Dp / 4) + c4], kv = k4[t * (Dp / 4) + c4], qv = q4[t * (Dp / 4) + c4];
+                const float4 kv = k4[t * (Dp / 4) + c4], qv = q4[t * (Dp / 4) + c4];
+                float4 gv = make_float4(dec, dec, dec, dec);
+                if constexpr (!HD) gv = g4[t * (Dp / 4) + c4];
                 const float g_[4] = {gv.x, gv.y, gv.z, gv.w}, k_[4] = {kv.x, kv.y, kv.z, kv.w}, q_[4] = {qv.x, qv.y, qv.z, qv.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -402,7 +436,7 @@ __global__ void __launch_bounds__(SCAN_J / (4 * NC) * 32, 2) delta_scan_kernel(c
             const float bt = betas[t], dot = qks[t];
 #pragma unroll
             for (int e = 0; e < NC; ++e) {
-                const float u = bt * (vs[t * SCAN_J + jl + e] - rk[e]);
+                const float u = bt * (vs[t * J + jl + e] - rk[e]);
 #pragma unroll
                 for (int c = 0; c < CH; ++c) st[e][c] = fmaf(kk[c], u, st[e][c]);
                 if (p == 0 && j + e < a.V) orow[(size_t)t * a.H * a.V + e] = fmaf(dot, u, rq[e]);
@@ -588,14 +622,21 @@ static int launch_ssd(const CcSeqSsdScan* a, cudaStream_t st) {
     return cuda_check("ssd_scan_kernel");
 }
 
+template <int CH, int NC, int TB, int J, bool HD>
+static int launch_delta_j(const CcSeqDeltaScan* a, cudaStream_t st) {
+    const size_t smem = sizeof(float) * 2 * (size_t)delta_buf_floats(DL_PARTS * (CH + 4), J, TB, HD);
+    static size_t configured = 48 * 1024;
+    auto kern = delta_scan_kernel<CH, NC, TB, J, HD>;
+    if (int rc = set_smem(kern, smem, configured)) return rc;
+    dim3 grid(a->H, (a->V + J - 1) / J);
+    kern<<<grid, J / (4 * NC) * 32, smem, st>>>(*a);
+    return cuda_check("delta_scan_kernel");
+}
+
 template <int CH, int NC, int TB>
 static int launch_delta(const CcSeqDeltaScan* a, cudaStream_t st) {
-    const size_t smem = sizeof(float) * 2 * (size_t)TB * (3 * DL_PARTS * (CH + 4) + SCAN_J + 2);
-    static size_t configured = 48 * 1024;
-    if (int rc = set_smem(delta_scan_kernel<CH, NC, TB>, smem, configured)) return rc;
-    dim3 grid(a->H, (a->V + SCAN_J - 1) / SCAN_J);
-    delta_scan_kernel<CH, NC, TB><<<grid, SCAN_J / (4 * NC) * 32, smem, st>>>(*a);
-    return cuda_check("delta_scan_kernel");
+    if (a->head_decay) return launch_delta_j<CH, NC, TB, SCAN_J, true>(a, st);
+    return launch_delta_j<CH, NC, TB, SCAN_J, false>(a, st);
 }
 
 }  // namespace ccn
@@ -658,7 +699,9 @@ int cc_seq_delta_prepare(const CcSeqDeltaScan* a, float* qn, float* kn, float* g
         a->T < 1 || a->H < 1 || a->G < 1 || a->H % a->G || a->D < 1 || a->prepared)
         return fail(CC_SEQ_ERR_INVALID_ARG, "delta_prepare: bad argument");
     const size_t warps = (size_t)a->T * a->H;
-    delta_prepare_kernel<<<(unsigned)((warps + 7) / 8), 256, 0, (cudaStream_t)stream>>>(*a, qn, kn, gd, beta, qk);
+    const unsigned blocks = (unsigned)((warps + 7) / 8);
+    if (a->head_decay) delta_prepare_kernel<true><<<blocks, 256, 0, (cudaStream_t)stream>>>(*a, qn, kn, gd, beta, qk);
+    else delta_prepare_kernel<false><<<blocks, 256, 0, (cudaStream_t)stream>>>(*a, qn, kn, gd, beta, qk);
     return cuda_check("delta_prepare_kernel");
 }
 

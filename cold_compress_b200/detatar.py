@@ -334,7 +334,9 @@ class RoutedExperts(nn.Module):
     `top` largest choices win and are weighted by their scores divided by their sum.  The last `identity` outputs are
     identity experts (the input itself).  A shared expert runs for every token, times sigmoid of one projection row.
     Its router, shared-gate and shared gate/up rows are part of the layer's fused projection of h.  Options: `scoring`
-    "sigmoid" scores every output on its own instead of the softmax; `group_top` makes a group's score the sum of its
+    "sigmoid" scores every output on its own instead of the softmax, "softmax_chosen" chooses by logit + correction (a
+    bias) and takes the softmax over the chosen logits as weights; `gated=False` makes an expert `down(act(up h))`;
+    `group_top` makes a group's score the sum of its
     that many largest choices instead of the largest; `renormalize=False` keeps the chosen scores as weights;
     `weight_scale` multiplies the weights; `shared_gate=False` adds the shared expert without a gate.
 
@@ -346,31 +348,35 @@ class RoutedExperts(nn.Module):
 
     def __init__(self, dim: int, n_experts: int, n_identity: int, ff: int, top: int, groups: int, keep: int,
                  shared_ff: int, act: int, dtype, scoring: str = "softmax", group_top: int = 1, renormalize: bool = True,
-                 weight_scale: float = 1.0, shared_gate: bool = True):
+                 weight_scale: float = 1.0, shared_gate: bool = True, gated: bool = True):
         super().__init__()
         self.dim, self.n_real, self.n_identity, self.ff, self.top = dim, int(n_experts), int(n_identity), int(ff), int(top)
         self.groups, self.keep, self.shared_ff, self.act = int(groups), int(keep), int(shared_ff), int(act)
         if (self.n_real + self.n_identity) % self.groups:
             raise ValueError("router outputs must split into equal groups")
-        if scoring not in ("softmax", "sigmoid"):
+        if scoring not in ("softmax", "sigmoid", "softmax_chosen"):
             raise ValueError(f"unknown router scoring {scoring!r}")
+        if not 1 <= self.top <= self.n_real + self.n_identity:
+            raise ValueError(f"a token cannot choose {self.top} of {self.n_real + self.n_identity} experts")
+        self.softmax_chosen, self.gated = scoring == "softmax_chosen", bool(gated)
         self.sigmoid_scores, self.group_top, self.renormalize = scoring == "sigmoid", int(group_top), bool(renormalize)
         self.weight_scale, self.sg_rows = float(weight_scale), (1 if shared_gate and self.shared_ff else 0)
         self.correction = _zeros(self.n_real + self.n_identity, dtype=torch.float32)
-        self.w_gu = _zeros(self.n_real, 2 * self.ff, dim, dtype=dtype)      # per expert: gate rows | up rows
+        # per expert: gate rows | up rows, or the up rows alone
+        self.w_gu = _zeros(self.n_real, (2 if self.gated else 1) * self.ff, dim, dtype=dtype)
         self.w_d = _zeros(self.n_real, dim, self.ff, dtype=dtype)
         self.w_shared_down = _zeros(dim, self.shared_ff, dtype=dtype) if self.shared_ff else None
 
     def n_rows(self):
         return self.n_real + self.n_identity + ((self.sg_rows + 2 * self.shared_ff) if self.shared_ff else 0)
 
-    def _route(self, hp: Tensor, off: int):
+    def route(self, hp: Tensor, off: int):
         T, dev = hp.shape[0], hp.device
         n = self.n_real + self.n_identity
         ids = torch.empty(T, self.top, dtype=torch.int32, device=dev)
         wts = torch.empty(T, self.top, dtype=torch.float32, device=dev)
         seq_ops.moe_route(hp[:, off:off + n], self.correction, ids, wts, self.groups, self.keep, self.top,
-                          self.sigmoid_scores, self.group_top, self.renormalize, self.weight_scale)
+                          self.sigmoid_scores, self.group_top, self.renormalize, self.weight_scale, self.softmax_chosen)
         return ids, wts
 
     def _few_tokens(self, h_act: Tensor, ids: Tensor):
@@ -388,7 +394,7 @@ class RoutedExperts(nn.Module):
     def one_token(self, hp: Tensor, off: int, h: Tensor, h_act: Tensor):
         """-> (jobs for the layer's closing launch, function that returns the result after it)."""
         n = self.n_real + self.n_identity
-        ids, wts = self._route(hp, off)
+        ids, wts = self.route(hp, off)
         y = self._few_tokens(h_act, ids)
         jobs, shared, sg = [], None, None
         if self.shared_ff:
@@ -399,8 +405,8 @@ class RoutedExperts(nn.Module):
 
     def forward(self, hp: Tensor, off: int, h: Tensor, h_act: Tensor, one_token_kernel: bool = True) -> Tensor:
         T, dev, dt = hp.shape[0], hp.device, self.w_gu.dtype
-        n, E, F, top = self.n_real + self.n_identity, self.dim, self.ff, self.top
-        ids, wts = self._route(hp, off)
+        n = self.n_real + self.n_identity
+        ids, wts = self.route(hp, off)
         shared = sg = None
         if self.shared_ff:
             g0 = off + n + self.sg_rows
@@ -408,29 +414,35 @@ class RoutedExperts(nn.Module):
             act = torch.empty(T, self.shared_ff, dtype=dt, device=dev)
             seq_ops.gated_unit(hp, g0, g0 + self.shared_ff, act, self.act)
             shared = _proj(act, self.w_shared_down)
-        M = T * top
-        if T <= self.small_t:
-            y, slot = self._few_tokens(h_act, ids), None
-        else:
-            counts = torch.empty(self.n_real, dtype=torch.int32, device=dev)
-            slot = torch.empty(M, dtype=torch.int32, device=dev)
-            perm = torch.empty(M, dtype=torch.int32, device=dev)
-            seq_ops.moe_group(ids, self.n_real, counts, slot, perm)
-            sizes = counts.tolist()
-            rows = sum(sizes)
-            y = torch.empty(max(rows, 1), E, dtype=torch.float32, device=dev)
-            if rows:
-                xs = torch.empty(rows, E, dtype=dt, device=dev)
-                seq_ops.gather_rows(h_act, perm, xs, rows)
-                lo = 0
-                for e, cnt in enumerate(sizes):
-                    if cnt:
-                        gu = _mm(xs[lo:lo + cnt], self.w_gu[e])
-                        act = torch.empty(cnt, F, dtype=dt, device=dev)
-                        seq_ops.gated_unit(gu, 0, F, act, self.act)
-                        y[lo:lo + cnt] = _mm(act, self.w_d[e])
-                        lo += cnt
+        slot, y = self.expert_rows(ids, h_act)
         return self._combine(ids, wts, slot, y, h, shared, sg)
+
+    def expert_rows(self, ids: Tensor, h_act: Tensor):
+        """(slot, y): the chosen real experts' outputs as fp32 rows of y, choice k of token t in row slot[t, k] (row
+        t * top + k when slot is None)."""
+        T, dev, dt = h_act.shape[0], h_act.device, self.w_gu.dtype
+        E, F, M = self.dim, self.ff, T * self.top
+        if T <= self.small_t:
+            return None, self._few_tokens(h_act, ids)
+        counts = torch.empty(self.n_real, dtype=torch.int32, device=dev)
+        slot = torch.empty(M, dtype=torch.int32, device=dev)
+        perm = torch.empty(M, dtype=torch.int32, device=dev)
+        seq_ops.moe_group(ids, self.n_real, counts, slot, perm)
+        sizes = counts.tolist()
+        rows = sum(sizes)
+        y = torch.empty(max(rows, 1), E, dtype=torch.float32, device=dev)
+        if rows:
+            xs = torch.empty(rows, E, dtype=dt, device=dev)
+            seq_ops.gather_rows(h_act, perm, xs, rows)
+            lo = 0
+            for e, cnt in enumerate(sizes):
+                if cnt:
+                    gu = _mm(xs[lo:lo + cnt], self.w_gu[e])
+                    act = torch.empty(cnt, F, dtype=dt, device=dev)
+                    seq_ops.gated_unit(gu, 0, F if self.gated else -1, act, self.act)
+                    _mm(act, self.w_d[e], out=y[lo:lo + cnt])
+                    lo += cnt
+        return slot, y
 
 
 # --------------------------------------------------------------------------------------------- a layer

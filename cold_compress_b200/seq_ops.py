@@ -328,14 +328,15 @@ def head_norm_gate(o, graw, nw, out, H, D, eps):
 
 
 def moe_route(logits, correction, ids, wts, groups, keep, top, sigmoid_scores=False, group_top=1, renormalize=True,
-              weight_scale=1.0):
-    """Router: softmax (or sigmoid) scores, choice = score + correction, the `keep` best of `groups` groups by the sum of
+              weight_scale=1.0, softmax_chosen=False):
+    """Router: softmax (or sigmoid) scores, choice = score + correction (softmax_chosen: choice = logit + correction, and
+    the weights are the softmax over the winners), the `keep` best of `groups` groups by the sum of
     their `group_top` largest choices, `top` winners; weights = winners' scores (renormalised or not) * weight_scale."""
     _need(("correction", correction, torch.float32), ("ids", ids, torch.int32), ("wts", wts, torch.float32))
     ptr, ld = _cols(_f32("logits", logits))
     T, n = logits.shape
     _lib.check_seq(_lib.load_seq().cc_seq_moe_route(ptr, ld, _p(correction), _p(ids), _p(wts), T, n, int(groups), int(keep), int(top),
-                                                    int(bool(sigmoid_scores)), int(group_top), int(bool(renormalize)),
+                                                    _lib.SCORE_CHOSEN if softmax_chosen else int(bool(sigmoid_scores)), int(group_top), int(bool(renormalize)),
                                                     float(weight_scale), _stream()), "cc_seq_moe_route")
 
 
@@ -352,13 +353,16 @@ def gather_rows(src, perm, dst, M):
 
 
 def moe_expert_tokens(wgu, wd, h, ids, act, y, kind):
-    """Experts of a few tokens, no grouping: wgu [n, 2F, E], wd [n, E, F], h [T, E], ids [T, top] -> y fp32 [T * top, E]."""
+    """Experts of a few tokens, no grouping: wgu [n, 2F, E] (or [n, F, E]: experts without a gate), wd [n, E, F], h [T, E],
+    ids [T, top], act [T * top, F] scratch -> y fp32 [T * top, E]."""
     _need(("wgu", wgu, None), ("wd", wd, wgu.dtype), ("h", h, wgu.dtype), ("ids", ids, torch.int32), ("act", act, wgu.dtype),
           ("y", y, torch.float32))
-    n, F2, E = wgu.shape
+    n, rows, E = wgu.shape
+    F = wd.shape[-1]
     T, top = ids.shape
+    assert rows in (F, 2 * F) and wd.shape == (n, E, F) and act.numel() == T * top * F
     _lib.check_seq(_lib.load_seq().cc_seq_moe_expert_tokens(_p(wgu), _p(wd), _p(h), _p(ids), _p(act), _p(y), _dt(wgu), T, top, n,
-                                                            F2 // 2, E, int(kind), _stream()), "cc_seq_moe_expert_tokens")
+                                                            F, E, int(kind), int(rows == 2 * F), _stream()), "cc_seq_moe_expert_tokens")
 
 
 def moe_combine(ids, wts, slot, y, h, shared, sg, out, n_real):
@@ -520,7 +524,7 @@ def ssd_scan(x, B, Cm, dt_raw, dt_bias, A_log, D, state, y, H, G, N, V):
 
 def delta_scan(q, k, v, beta_raw, a_raw, dt_bias, A_log, state, o, H, G, D, V, q_scale, unit_eps=1e-6):
     """Delta rule with a decay per key channel over T tokens: q / k [T, G*D], v [T, H*V], beta_raw [T, H], a_raw
-    [T, H*D] (fp32 column ranges), state fp32 [H, D, V] carried, o fp32 [T, H*V]."""
+    [T, H*D] (or [T, H]: one decay per head; fp32 column ranges), state fp32 [H, D, V] carried, o fp32 [T, H*V]."""
     _need(("dt_bias", dt_bias, torch.float32), ("A_log", A_log, torch.float32), ("state", state, torch.float32), ("o", o, torch.float32))
     a = _lib.CcSeqDeltaScan()
     a.q, a.ldqk = _cols(_f32("q", q))
@@ -528,7 +532,11 @@ def delta_scan(q, k, v, beta_raw, a_raw, dt_bias, A_log, state, o, H, G, D, V, q
     a.v, a.ldv = _cols(_f32("v", v))
     a.beta_raw, a.ldb = _cols(_f32("beta_raw", beta_raw))
     a.a_raw, a.lda = _cols(_f32("a_raw", a_raw))
-    assert ldk == a.ldqk and state.numel() == H * D * V and o.shape == (q.shape[0], H * V) and dt_bias.numel() == H * D
+    per_head = a_raw.shape[1] == H and dt_bias.numel() == H
+    gate_cols = H if per_head else H * D
+    assert ldk == a.ldqk and state.numel() == H * D * V and o.shape == (q.shape[0], H * V)
+    assert dt_bias.numel() == gate_cols and a_raw.shape[1] == gate_cols
+    a.head_decay = int(per_head)
     a.dt_bias, a.A_log, a.state, a.o = _p(dt_bias), _p(A_log), _p(state), _p(o)
     a.T, a.H, a.G, a.D, a.V = q.shape[0], int(H), int(G), int(D), int(V)
     a.q_scale, a.unit_eps = float(q_scale), float(unit_eps)
@@ -537,10 +545,11 @@ def delta_scan(q, k, v, beta_raw, a_raw, dt_bias, A_log, state, o, H, G, D, V, q
         # long steps: the per-token preparation (unit vectors, decays, beta) in a launch of its own, spread over the GPU,
         # instead of once per column tile inside the scan; same arithmetic, same bits
         f32 = dict(dtype=torch.float32, device=o.device)
-        qn, kn, gd = (torch.empty(a.T, H * D, **f32) for _ in range(3))
+        qn, kn = (torch.empty(a.T, H * D, **f32) for _ in range(2))
+        gd = torch.empty(a.T, gate_cols, **f32)
         bt, qk = torch.empty(a.T, H, **f32), torch.empty(a.T, H, **f32)
         _lib.check_seq(lib.cc_seq_delta_prepare(C.byref(a), _p(qn), _p(kn), _p(gd), _p(bt), _p(qk), _stream()), "cc_seq_delta_prepare")
-        a.q, a.k, a.ldqk, a.a_raw, a.lda, a.beta_raw, a.ldb = _p(qn), _p(kn), H * D, _p(gd), H * D, _p(bt), H
+        a.q, a.k, a.ldqk, a.a_raw, a.lda, a.beta_raw, a.ldb = _p(qn), _p(kn), H * D, _p(gd), gate_cols, _p(bt), H
         a.qk, a.G, a.prepared = _p(qk), int(H), 1
     _lib.check_seq(lib.cc_seq_delta_scan(C.byref(a), _stream()), "cc_seq_delta_scan")
 
@@ -635,3 +644,25 @@ def poly_norm(src, coef, out, eps):
     T, F = out.shape
     assert src.shape == (T, F) and coef.numel() == 4
     _lib.check_seq(_lib.load_seq().cc_seq_poly_norm(ptr, ld, _p(coef), _p(out), _dt(out), T, F, float(eps), _stream()), "cc_seq_poly_norm")
+
+
+# ------------------------------------------------------------------------------------------------------------------
+# Fifth part of the C ABI (csrc/seq/post_kernels.cu): sublayer outputs that are normed before they join the stream.
+
+def post_norm(x, y, w, eps, gain_offset=0.0, wts=None, slot=None, x_out=None, x_act=None, next_w=None, next_eps=0.0,
+              next_offset=0.0):
+    """x (fp32 [T, E]) + rms_norm(r) * (w + gain_offset) -> x_out (default: x in place), with r the row of y [T, E] or,
+    with wts [T, top], the weighted sum of the rows slot[t, k] (default t * top + k) of y [*, E].  x_act: the sum in the
+    compute dtype, or the RMS norm of it with gain next_w + next_offset."""
+    _need(("x", x, torch.float32), ("w", w, torch.float32), ("wts", wts, torch.float32), ("slot", slot, torch.int32),
+          ("x_out", x_out, torch.float32), ("x_act", x_act, None), ("next_w", next_w, torch.float32))
+    a = _lib.CcSeqPostNorm()
+    T, E = x.shape
+    a.y, a.ldy = _cols(_f32("y", y))
+    assert y.shape[1] == E and w.numel() == E and (x_act is None or x_act.shape == (T, E)) and (x_out is None or x_out.shape == (T, E))
+    assert (y.shape[0] == T) if wts is None else (wts.shape[0] == T and a.ldy == E and (slot is not None or y.shape[0] >= wts.numel()))
+    a.x, a.wts, a.slot, a.top = _p(x), _p(wts), _p(slot), 0 if wts is None else wts.shape[1]
+    a.w, a.eps, a.gain_offset, a.x_out = _p(w), float(eps), float(gain_offset), _p(x_out)
+    a.x_act, a.act_dtype = _p(x_act), _dt(x_act) if x_act is not None else _lib.DT_F32
+    a.next_w, a.next_eps, a.next_offset, a.T, a.E = _p(next_w), float(next_eps), float(next_offset), T, E
+    _lib.check_seq(_lib.load_seq().cc_seq_post_norm(C.byref(a), _stream()), "cc_seq_post_norm")

@@ -213,28 +213,34 @@ class BlockRotaryAttention(nn.Module):
 
 
 class GatedDeltaRule(nn.Module):
-    """Delta rule with a decay per key channel.  q, k (kv_heads x dim) and v (heads x v_dim) pass short convolutions with
-    silu; q and k become unit vectors per head (q also times dim^-1/2); `beta = sigmoid(W_b h)` per head; decay
-    `g = exp(-exp(A_log) * softplus(W_a2 W_a1 h + dt_bias))` per head and key channel; per head `S <- diag(g) S;
+    """Delta rule with decay.  q, k (kv_heads x dim) and v (heads x v_dim) pass short convolutions with silu; q and k
+    become unit vectors per head (q also times dim^-1/2); `beta = sigmoid(W_b h)` per head; decay
+    `g = exp(-exp(A_log) * softplus(d + dt_bias))` per head and key channel with the low-rank projection
+    `d = W_a2 W_a1 h`, or (`decay_rank` None) one per head with `d = W_a h`; per head `S <- diag(g) S;
     u = beta (v - S^T k); S <- S + k u^T; o = S^T q`; o is RMS-normed per head with a gain shared by the heads and
-    multiplied by `sigmoid(W_g2 W_g1 h)`.  Input rows [q | k | v | b | a1 | g1] are part of the owner's fused projection.
-    State per sequence: the convolution tail and S [heads, dim, v_dim] (fp32)."""
+    multiplied by `gate_act(W_g2 W_g1 h)` or (`gate_rank` None) `gate_act(W_g h)`.  Input rows [q | k | v | b | a1 | g1]
+    (or [.. | a | g]) are part of the owner's fused projection.  State per sequence: the convolution tail and S
+    [heads, dim, v_dim] (fp32)."""
 
     unit_eps = 1e-6
 
-    def __init__(self, dim: int, heads: int, kv_heads: int, head_dim: int, v_dim: int, taps: int, decay_rank: int, gate_rank: int,
-                 eps: float, dtype):
+    def __init__(self, dim: int, heads: int, kv_heads: int, head_dim: int, v_dim: int, taps: int, decay_rank: Optional[int],
+                 gate_rank: Optional[int], eps: float, dtype, gate_act: int = _lib.ACT_SIGMOID):
         super().__init__()
         if heads % kv_heads:
             raise ValueError("kv heads must divide the heads")
         self.dim, self.heads, self.kv_heads, self.head_dim, self.v_dim = dim, int(heads), int(kv_heads), int(head_dim), int(v_dim)
-        self.decay_rank, self.gate_rank, self.eps = int(decay_rank), int(gate_rank), float(eps)
+        self.decay_rank = None if decay_rank is None else int(decay_rank)
+        self.gate_rank = None if gate_rank is None else int(gate_rank)
+        self.eps, self.gate_act = float(eps), int(gate_act)
         self.conv_width = 2 * self.kv_heads * self.head_dim + self.heads * self.v_dim
-        self.in_rows = self.conv_width + self.heads + self.decay_rank + self.gate_rank
+        self.a_rows = self.heads if self.decay_rank is None else self.decay_rank
+        self.g_rows = self.heads * self.v_dim if self.gate_rank is None else self.gate_rank
+        self.in_rows = self.conv_width + self.heads + self.a_rows + self.g_rows
         self.conv = ShortConv(self.conv_width, taps, act=_lib.ACT_SILU)
-        self.w_a2 = _zeros(self.heads * self.head_dim, self.decay_rank, dtype=dtype)
-        self.w_g2 = _zeros(self.heads * self.v_dim, self.gate_rank, dtype=dtype)
-        self.dt_bias = _zeros(self.heads * self.head_dim, dtype=torch.float32)
+        self.w_a2 = None if self.decay_rank is None else _zeros(self.heads * self.head_dim, self.decay_rank, dtype=dtype)
+        self.w_g2 = None if self.gate_rank is None else _zeros(self.heads * self.v_dim, self.gate_rank, dtype=dtype)
+        self.dt_bias = _zeros(self.heads * (1 if self.decay_rank is None else self.head_dim), dtype=torch.float32)
         self.A_log = _zeros(self.heads, dtype=torch.float32)
         self.norm_w = _zeros(self.v_dim, dtype=torch.float32)
         self.w_o = _zeros(dim, self.heads * self.v_dim, dtype=dtype)
@@ -243,26 +249,35 @@ class GatedDeltaRule(nn.Module):
         return dict(n_heads=self.heads, head_dim=self.head_dim, state_cols=self.v_dim, state_vectors=self.conv.taps - 1,
                     state_width=self.conv_width)
 
+    def _second_products(self, hp: Tensor, oa: int, og: int, one_token: bool):
+        """The decay and gate rows: columns of the fused projection, or products of its low-rank columns."""
+        T, dev, dt = hp.shape[0], hp.device, self.w_o.dtype
+        outs, jobs = [], []
+        for off, n, w in ((oa, self.a_rows, self.w_a2), (og, self.g_rows, self.w_g2)):
+            if w is None:
+                outs.append(hp[:, off:off + n])
+            elif one_token and T == 1:
+                outs.append(_out(w))
+                jobs.append((hp[:, off:off + n], w, outs[-1]))
+            else:
+                low = torch.empty(T, n, dtype=dt, device=dev)
+                seq_ops.gated_unit(hp, off, -1, low, _lib.ACT_NONE)
+                outs.append(_mm(low, w))
+        if jobs:
+            seq_ops.gemv_multi(jobs)
+        return outs
+
     def core(self, hp: Tensor, off: int, ip: Tensor, state, one_token: bool) -> Tensor:
         T, dev, dt = hp.shape[0], hp.device, self.w_o.dtype
         H, G, D, V = self.heads, self.kv_heads, self.head_dim, self.v_dim
         ob = off + self.conv_width
-        oa, og = ob + H, ob + H + self.decay_rank
         c = self.conv(hp[:, off:off + self.conv_width], state.vectors)
-        if one_token and T == 1:
-            a_raw, g_raw = _out(self.w_a2), _out(self.w_g2)
-            seq_ops.gemv_multi([(hp[:, oa:oa + self.decay_rank], self.w_a2, a_raw), (hp[:, og:og + self.gate_rank], self.w_g2, g_raw)])
-        else:
-            low_a = torch.empty(T, self.decay_rank, dtype=dt, device=dev)
-            low_g = torch.empty(T, self.gate_rank, dtype=dt, device=dev)
-            seq_ops.gated_unit(hp, oa, -1, low_a, _lib.ACT_NONE)
-            seq_ops.gated_unit(hp, og, -1, low_g, _lib.ACT_NONE)
-            a_raw, g_raw = _mm(low_a, self.w_a2), _mm(low_g, self.w_g2)
+        a_raw, g_raw = self._second_products(hp, ob + H, ob + H + self.a_rows, one_token)
         o = torch.empty(T, H * V, dtype=torch.float32, device=dev)
         seq_ops.delta_scan(c[:, :G * D], c[:, G * D:2 * G * D], c[:, 2 * G * D:], hp[:, ob:ob + H], a_raw, self.dt_bias, self.A_log,
                            state.matrix, o, H, G, D, V, D ** -0.5, self.unit_eps)
         on = torch.empty(T, H * V, dtype=dt, device=dev)
-        seq_ops.gated_rms_groups(o, g_raw, _lib.ACT_SIGMOID, False, self.norm_w, on, H, self.eps)
+        seq_ops.gated_rms_groups(o, g_raw, self.gate_act, False, self.norm_w, on, H, self.eps)
         return on
 
 
@@ -548,6 +563,7 @@ class TefovikTransformer(nn.Module):
                 if (r.decay_rank, r.gate_rank) != (ra, rg):     # the ranks come from the tensors
                     dev, dt = r.w_a2.device, r.w_a2.dtype
                     r.decay_rank, r.gate_rank = ra, rg
+                    r.a_rows, r.g_rows = ra, rg
                     r.in_rows = r.conv_width + r.heads + ra + rg
                     r.w_a2 = _zeros(r.heads * r.head_dim, ra, dtype=dt).to(dev)
                     r.w_g2 = _zeros(rv, rg, dtype=dt).to(dev)

@@ -30,11 +30,14 @@ from . import _lib, seq_ops
 from .cache import get_cache_constructor
 
 
-def _mm(a: Tensor, w: Tensor) -> Tensor:
-    """a [T, K] @ w[N, K]^T -> fp32 [T, N]: cuBLAS with fp32 accumulation and fp32 output in both compute dtypes."""
+def _mm(a: Tensor, w: Tensor, out: Optional[Tensor] = None) -> Tensor:
+    """a [T, K] @ w[N, K]^T -> fp32 [T, N] (into `out` when given): cuBLAS with fp32 accumulation and fp32 output in both
+    compute dtypes."""
     if a.dtype == torch.float32:
-        return torch.mm(a, w.t())
-    return torch.mm(a, w.t(), out_dtype=torch.float32)
+        return torch.mm(a, w.t()) if out is None else torch.mm(a, w.t(), out=out)
+    if out is None:
+        return torch.mm(a, w.t(), out_dtype=torch.float32)
+    return torch.mm(a, w.t(), out_dtype=torch.float32, out=out)
 
 
 # --------------------------------------------------------------------------------------------- configuration

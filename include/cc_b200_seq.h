@@ -21,7 +21,7 @@
 extern "C" {
 #endif
 
-#define CC_SEQ_ABI_VERSION 4
+#define CC_SEQ_ABI_VERSION 5
 
 #define CC_SEQ_OK                     0
 #define CC_SEQ_ERR_INVALID_ARG       -1
@@ -300,16 +300,21 @@ int cc_seq_head_norm_gate(const float* o, const float* graw, int64_t ldg, const 
                           int32_t T, int32_t H, int32_t D, float eps, void* stream);
 
 /*
- * Router of a mixture of experts over n outputs (real and identity experts alike), logits fp32 [T, ld]:
- * scores s = softmax(logits) over all outputs, or sigmoid(logits) each on its own (`sigmoid_scores`); choice = s +
- * correction; the outputs form `groups` equal groups of neighbours and only those of the `keep` groups with the largest
+ * Router of a mixture of experts over n outputs (real and identity experts alike), logits fp32 [T, ld].  `scoring`:
+ * CC_SCORE_SOFTMAX  s = softmax(logits) over all outputs, choice = s + correction;
+ * CC_SCORE_SIGMOID  s = sigmoid(logits) each on its own, choice = s + correction;
+ * CC_SCORE_CHOSEN   choice = logits + correction (a bias), and the weights are the softmax over the winners' choices.
+ * The outputs form `groups` equal groups of neighbours and only those of the `keep` groups with the largest
  * group score can be chosen (the others count as minus infinity), a group's score being the sum of its `group_top`
  * largest choices (1 = its maximum); the `top` largest choices win (the lower index on a tie);
- * wts = s of the winners / (their sum + 1e-20) when `renormalize`, else s; both times weight_scale.
- * ids int32 [T, top], wts fp32 [T, top].
+ * wts = s of the winners / (their sum + 1e-20) when `renormalize`, else s (CC_SCORE_CHOSEN: the softmax, whatever
+ * `renormalize` says); all times weight_scale.  ids int32 [T, top], wts fp32 [T, top].
  */
+#define CC_SCORE_SOFTMAX 0
+#define CC_SCORE_SIGMOID 1
+#define CC_SCORE_CHOSEN  2
 int cc_seq_moe_route(const float* logits, int64_t ld, const float* correction, int32_t* ids, float* wts, int32_t T,
-                     int32_t n, int32_t groups, int32_t keep, int32_t top, int32_t sigmoid_scores, int32_t group_top,
+                     int32_t n, int32_t groups, int32_t keep, int32_t top, int32_t scoring, int32_t group_top,
                      int32_t renormalize, float weight_scale, void* stream);
 
 /* Groups the M = T * top (token, choice) pairs by real expert (id < n_real): counts [n_real], slot [M] = row of the
@@ -319,10 +324,11 @@ int cc_seq_moe_group(const int32_t* ids, int32_t M, int32_t top, int32_t n_real,
 int cc_seq_gather_rows(const void* src, const int32_t* perm, void* dst, int32_t dtype, int32_t M, int32_t E, void* stream);
 
 /* Experts for a few tokens without grouping: pair m = t * top + k with expert e = ids[m] < n_real:
- * act[m] = act(Wgu[e, 0:F] h[t]) * (Wgu[e, F:2F] h[t]),  y[m] = Wd[e] act[m]  (fp32 [M, E]).  Weights, h and act in dtype. */
+ * act[m] = act(Wgu[e, 0:F] h[t]) * (Wgu[e, F:2F] h[t]),  y[m] = Wd[e] act[m]  (fp32 [M, E]).  Weights, h and act in dtype.
+ * gated == 0: the experts have F input rows only and act[m] = act(Wgu[e, 0:F] h[t]). */
 int cc_seq_moe_expert_tokens(const void* Wgu, const void* Wd, const void* h, const int32_t* ids, void* act, float* y,
                              int32_t dtype, int32_t T, int32_t top, int32_t n_real, int32_t F, int32_t E, int32_t kind,
-                             void* stream);
+                             int32_t gated, void* stream);
 
 /* out[t] = sum_k wts[t, k] * (ids[t, k] < n_real ? y[slot[t, k]] : h[t]) + sigmoid(sg[t * ld_sg]) * shared[t];
  * slot == NULL means row t * top + k; shared may be NULL; sg == NULL means no gate on it; h may be NULL when there are
@@ -396,12 +402,13 @@ typedef struct CcSeqSsdScan {
 int cc_seq_ssd_scan(const CcSeqSsdScan* a, void* stream);
 
 /*
- * Delta rule with a decay per key channel, one state S [D, V] per head (head h reads q / k head h / (H / G)):
+ * Delta rule with a decay per key channel (or, with head_decay, one decay per head), one state S [D, V] per head (head h reads q / k head h / (H / G)):
  *   qn = q / sqrt(sum(q^2) + unit_eps) * q_scale;  kn = k / sqrt(sum(k^2) + unit_eps);  beta = sigmoid(beta_raw)
  *   g[i] = exp(-exp(A_log[h]) * softplus(a_raw[h * D + i] + dt_bias[h * D + i]))
+ *   (head_decay: g[i] = exp(-exp(A_log[h]) * softplus(a_raw[h] + dt_bias[h])) for every i)
  *   S <- diag(g) S;  u = beta * (v - S^T kn);  S <- S + kn u^T;  o = S^T qn
  * q, k fp32 [T, ldqk] (G * D columns), v fp32 [T, ldv] (H * V), beta_raw fp32 [T, ldb] (H), a_raw fp32 [T, lda]
- * (H * D), o fp32 [T, H * V] contiguous, state fp32 [H, D, V] read and written.  Exactly sequential in t.
+ * (H * D columns; H with head_decay), o fp32 [T, H * V] contiguous, state fp32 [H, D, V] read and written.  Exactly sequential in t.
  */
 typedef struct CcSeqDeltaScan {
     const float* q;  const float* k;  int64_t ldqk;
@@ -416,10 +423,11 @@ typedef struct CcSeqDeltaScan {
      * qk [T, H] holds qn . kn, all as cc_seq_delta_prepare writes them; the scan then only runs the recurrence. */
     const float* qk;
     int32_t prepared;
+    int32_t head_decay;
 } CcSeqDeltaScan;
 int cc_seq_delta_scan(const CcSeqDeltaScan* a, void* stream);
-/* The per-token preparation of cc_seq_delta_scan alone, spread over the GPU: qn, kn, gd fp32 [T, H * D], beta, qk fp32
- * [T, H], from an unprepared argument block.  Worth its launch for long steps; gives the same bits as the scan's own. */
+/* The per-token preparation of cc_seq_delta_scan alone, spread over the GPU: qn, kn, gd fp32 [T, H * D] (gd [T, H] with
+ * head_decay), beta, qk fp32 [T, H], from an unprepared argument block.  Worth its launch for long steps; gives the same bits as the scan's own. */
 int cc_seq_delta_prepare(const CcSeqDeltaScan* a, float* qn, float* kn, float* gd, float* beta, float* qk, void* stream);
 
 /*
@@ -511,6 +519,29 @@ int cc_seq_qk_row_norm(const CcSeqQkRowNorm* a, void* stream);
  * element, N(u) = u / sqrt(mean(u^2) + eps) over the F columns; coef fp32 [4] on the device; out [T, F] in out_dtype. */
 int cc_seq_poly_norm(const float* in, int64_t ld, const float* coef, void* out, int32_t out_dtype, int32_t T, int32_t F,
                      float eps, void* stream);
+
+/* ------------------------------------------------------------------------------------------------------------------
+ * Fifth part (csrc/seq/post_kernels.cu): sublayers whose OUTPUT is normed before it joins the stream.
+ * ------------------------------------------------------------------------------------------------------------------ */
+
+/*
+ * Per row t of the fp32 stream x [T, E]:
+ *   r = y[t]                                                             (top == 0; y fp32 [T, ldy])
+ *     = sum_k wts[t, k] * y[slot ? slot[t * top + k] : t * top + k]      (top  > 0; y fp32 rows of E, wts fp32 [T, top])
+ *   s = x[t] + r / sqrt(mean(r^2) + eps) * (w + gain_offset);   x_out[t] = s       (x_out NULL: in place)
+ *   x_act[t] = s, or with next_w:  s / sqrt(mean(s^2) + next_eps) * (next_w + next_offset), in act_dtype (x_act may be NULL)
+ */
+typedef struct CcSeqPostNorm {
+    float* x;
+    const float* y;  int64_t ldy;
+    const float* wts;  const int32_t* slot;  int32_t top;
+    const float* w;  float eps, gain_offset;
+    float* x_out;
+    void* x_act;  int32_t act_dtype;
+    const float* next_w;  float next_eps, next_offset;
+    int32_t T, E;
+} CcSeqPostNorm;
+int cc_seq_post_norm(const CcSeqPostNorm* a, void* stream);
 
 #ifdef __cplusplus
 }
