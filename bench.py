@@ -825,6 +825,38 @@ def _nevodra_model(sz, extra, device, dtype):
     return model.eval()
 
 
+NOBODRA_EXPERT_FF = {"1b": 2560, "8b": 4480}     # 16 experts, 4 chosen, no gate: as many active rows as the Nevodra arm has on average
+
+
+def _nobodra_config(sz, ff):
+    """Delta-rule layers (half as many heads of 128 x 128 as the shape has, taps 4; the same state as the Tefovik arm's)
+    alternate with windowed attention (the shape's heads and window, half of each head rotated, values = keys); every layer
+    has 16 ungated experts, 4 chosen."""
+    E, D = sz["width"], sz["head"]
+    delta = {"heads": sz["heads"] // 2, "kv_heads": sz["heads"] // 2, "dim": 128, "vdim": 128, "conv": 4}
+    window = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": sz["window"]},
+              "rot": {"base": 1000000.0, "dims": D // 2}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 16, "top": 4}}
+    layers = [{"type": "delta" if i % 2 == 0 else "attention", "mixer": delta if i % 2 == 0 else window, "mlp": moe} for i in range(sz["layers"])]
+    return {"architecture": "Nobodra", "vocab": sz["vocab"], "width": E, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def _nobodra_model(sz, ff, device, dtype):
+    from cold_compress_b200.nobodra import NobodraTransformer
+    with torch.device(device):
+        model = NobodraTransformer.from_config(_nobodra_config(sz, ff), dtype)
+    gen = torch.Generator(device=device).manual_seed(0)
+    with torch.no_grad():
+        for name, p in model.named_parameters():
+            if name.endswith("conv.weight"):
+                p.fill_(1.0 / p.shape[1])
+            elif p.dim() >= 2:
+                p.copy_(torch.empty(p.shape, device=device).normal_(0.0, 0.02, generator=gen))
+            elif name.endswith(("q_norm", "k_norm", "norm_w")):
+                p.fill_(1.0)
+    return model.eval()
+
+
 def _llama_model(sz, device):
     from cold_compress_b200.model import ModelArgs, Transformer
     cfg = ModelArgs(block_size=sz["prompt"] + 1024, vocab_size=sz["vocab"], n_layer=sz["layers"], n_head=sz["heads"],
@@ -869,7 +901,7 @@ def run_design(args):
     flush = torch.zeros(64 << 20, dtype=torch.float32, device=device)
     rows = []
     arms = {"detatar": ("detatar", "tidelorn"), "tefovik": ("tefovik", "detatar"),
-            "nevodra": ("nevodra", "detatar")}.get(args.design_model, ("tidelorn", "llama"))
+            "nevodra": ("nevodra", "detatar"), "nobodra": ("nobodra", "nevodra")}.get(args.design_model, ("tidelorn", "llama"))
     for name in names:
         sz = DESIGN_SIZES[name]
         P = sz["prompt"]
@@ -879,6 +911,7 @@ def run_design(args):
             model = (_detatar_model(sz, DETATAR_SIZES[name], device, torch.bfloat16) if arm == "detatar" else
                      _nevodra_model(sz, DETATAR_SIZES[name], device, torch.bfloat16) if arm == "nevodra" else
                      _tefovik_model(sz, device, torch.bfloat16) if arm == "tefovik" else
+                     _nobodra_model(sz, NOBODRA_EXPERT_FF[name], device, torch.bfloat16) if arm == "nobodra" else
                      _tidelorn_model(sz, device, torch.bfloat16) if arm == "tidelorn" else _llama_model(sz, device))
             ck = cache_kwargs(dict(slots=1.0, pattern="tile", strategy="full", compressor="recent_global"))
             ck["global_tokens"] = 0
@@ -912,9 +945,10 @@ def run_design(args):
                 torch.cuda.synchronize()
                 dms = a.elapsed_time(b) / args.steps
             wbytes = sum(p.numel() * p.element_size() for n, p in model.named_parameters() if p.dim() >= 2 and "tok_embeddings" not in n and "bigram" not in n)
-            if arm in ("detatar", "nevodra"):      # a token reads `top` experts of each mixture, not all of them, and one copy of W_uk
+            if arm in ("detatar", "nevodra", "nobodra"):      # a token reads `top` experts of each mixture, not all of them, and one copy of W_uk
                 for layer in model.layers:
-                    f, m = layer.block.mlp, layer.block.mixer
+                    block = getattr(layer, "block", layer)
+                    f, m = block.mlp, block.mixer
                     if hasattr(f, "w_gu"):
                         wbytes -= (f.n_real - f.top) * (f.w_gu[0].numel() + f.w_d[0].numel()) * f.w_gu.element_size()
                     if hasattr(m, "w_uk_t"):
@@ -926,14 +960,18 @@ def run_design(args):
             del model, decoder
             torch.cuda.empty_cache()
         row["kernels"] = _design_kernels(sz, device, hbm)
-        if args.design_model in ("detatar", "tefovik", "nevodra"):
+        if args.design_model in ("detatar", "tefovik", "nevodra", "nobodra"):
             row["detatar_kernels"] = _detatar_kernels(sz, DETATAR_SIZES[name], device, hbm)
         if args.design_model == "nevodra":
             row["nevodra_kernels"] = _nevodra_kernels(sz, DETATAR_SIZES[name], device, hbm)
-        if args.design_model == "tefovik":
+        if args.design_model == "nobodra":
+            row["nevodra_kernels"] = _nevodra_kernels(sz, DETATAR_SIZES[name], device, hbm)
+            row["nobodra_kernels"] = _nobodra_kernels(sz, NOBODRA_EXPERT_FF[name], device, hbm)
+        if args.design_model in ("tefovik", "nobodra"):
             row["tefovik_kernels"] = _tefovik_kernels(sz, device, hbm)
         rows.append(row)
-    metric = ("prefill and decode tokens/s, Nevodra beside Detatar at equal layer shape" if args.design_model == "nevodra" else
+    metric = ("prefill and decode tokens/s, Nobodra beside Nevodra at equal layer shape" if args.design_model == "nobodra" else
+              "prefill and decode tokens/s, Nevodra beside Detatar at equal layer shape" if args.design_model == "nevodra" else
               "prefill and decode tokens/s, Detatar beside Tidelorn at equal layer shape" if args.design_model == "detatar" else
               "prefill and decode tokens/s, Tefovik beside Detatar at equal layer shape" if args.design_model == "tefovik" else
               "prefill and decode tokens/s, Tidelorn beside Llama (full cache) at equal layer shape")
@@ -1206,6 +1244,66 @@ def _nevodra_kernels(sz, extra, device, hbm):
     return out
 
 
+def _nobodra_kernels(sz, ff, device, hbm):
+    """The Nobodra kernels alone at this shape: the delta-rule scan with one decay per head over a prompt and for one token,
+    the output norm + sum (with and without the experts' weighted sum) over a prompt and for one token, the q / k rows of
+    the windowed attention, and the chosen ungated experts of one token.  (The windowed attention itself is
+    `prefill_attention_window` / `decode_attention_window`.)"""
+    from cold_compress_b200 import _lib, seq_ops
+    cfg = _nobodra_config(sz, ff)
+    P, E = sz["prompt"], sz["width"]
+    gen = torch.Generator(device=device).manual_seed(6)
+    out = {}
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=device)
+
+    def token_us(fn, n=20, flush=None):
+        fn(0)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(n):
+                fn(i)
+        return _time_events(graph.replay, 2, 5, flush) * 1e3 / n
+
+    def rate(nbytes, us):
+        return {"us": round(us, 2), "gb_per_s": round(nbytes / us / 1e3, 1), "frac_of_hbm": round(nbytes / us / 1e3 / hbm, 3)}
+
+    m = cfg["layers"][0]["mixer"]
+    H, D, V = m["heads"], m["dim"], m["vdim"]
+    q, k = (torch.randn(P, H * D, device=device, generator=gen) for _ in range(2))
+    v = torch.randn(P, H * V, device=device, generator=gen) * 0.1
+    a_raw, beta = torch.randn(P, H, device=device, generator=gen), torch.randn(P, H, device=device, generator=gen)
+    dtb, alog = torch.zeros(H, device=device), torch.zeros(H, device=device)
+    state, o = torch.zeros(H, D, V, device=device), torch.empty(P, H * V, device=device)
+    scan = lambda n: seq_ops.delta_scan(q[:n], k[:n], v[:n], beta[:n], a_raw[:n], dtb, alog, state, o[:n], H, H, D, V, D ** -0.5)
+    ms = _time_events(lambda: scan(P), 2, 3)
+    out["delta_rule_scan_head_decay_prompt"] = {"ms": round(ms, 3), "fp32_tflops": round(7.0 * P * H * D * V / ms / 1e9, 2),
+                                                "gb_per_s": round((2.0 * H * D + 2 * H * V + 2 * H) * P * 4 / ms / 1e6, 1)}
+    out["delta_rule_scan_head_decay_token"] = rate(2 * H * D * V * 4, token_us(lambda i: scan(1)))
+    x, y = torch.randn(P, E, device=device, generator=gen), torch.randn(P, E, device=device, generator=gen)
+    w, act = torch.zeros(E, device=device), torch.empty(P, E, device=device, dtype=torch.bfloat16)
+    us = 1e3 * _time_events(lambda: seq_ops.post_norm(x, y, w, 1e-5, 1.0, x_act=act), 2, 3, flush)
+    out["output_norm_prompt"] = rate(P * E * (3 * 4 + 2), us)          # y read, x read and written, bf16 copy written
+    out["output_norm_token"] = {"us": round(token_us(lambda i: seq_ops.post_norm(x[:1], y[:1], w, 1e-5, 1.0, x_act=act[:1])), 2)}
+    top = cfg["layers"][0]["mlp"]["router"]["top"]
+    rows = torch.randn(P * top, E, device=device, generator=gen)
+    wts = torch.full((P, top), 1.0 / top, device=device)
+    slot = torch.randperm(P * top, device=device, generator=gen).to(torch.int32)
+    us = 1e3 * _time_events(lambda: seq_ops.post_norm(x, rows, w, 1e-5, 1.0, wts=wts, slot=slot, x_act=act), 2, 3, flush)
+    out["expert_sum_output_norm_prompt"] = rate(P * E * ((2 + top) * 4 + 2), us)
+    out["expert_sum_output_norm_token"] = {"us": round(token_us(lambda i: seq_ops.post_norm(x[:1], rows[:top], w, 1e-5, 1.0, wts=wts[:1], x_act=act[:1])), 2)}
+    del rows
+    n = cfg["layers"][0]["mlp"]["router"]["experts"]
+    wu = (torch.randn(n, ff, E, device=device, generator=gen) * 0.02).to(torch.bfloat16)
+    wd = (torch.randn(n, E, ff, device=device, generator=gen) * 0.02).to(torch.bfloat16)
+    h = torch.randn(1, E, device=device, generator=gen).to(torch.bfloat16)
+    picks = [(torch.arange(top, dtype=torch.int32, device=device) * 4 + i).view(1, top) % n for i in range(4)]   # other experts each time
+    eact, ey = torch.empty(top, ff, device=device, dtype=torch.bfloat16), torch.empty(top, E, device=device)
+    us = token_us(lambda i: seq_ops.moe_expert_tokens(wu, wd, h, picks[i], eact, ey, _lib.ACT_RELU_SQ), 4, flush)
+    out["experts_token"] = rate(top * 2 * ff * E * 2, us)
+    return out
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1218,9 +1316,9 @@ def main():
     ap.add_argument("--design", default="", metavar="SIZES",
                     help="instead of the headline workload: Tidelorn beside the Llama-family model at equal layer shape, "
                          "comma-separated sizes of " + "/".join(DESIGN_SIZES))
-    ap.add_argument("--design-model", default="tidelorn", choices=["tidelorn", "detatar", "tefovik", "nevodra"],
+    ap.add_argument("--design-model", default="tidelorn", choices=["tidelorn", "detatar", "tefovik", "nevodra", "nobodra"],
                     help="with --design: which design is measured (tidelorn: beside the Llama-family model; detatar: beside "
-                         "Tidelorn; tefovik, nevodra: beside Detatar; sizes " + "/".join(DETATAR_SIZES) + ")")
+                         "Tidelorn; tefovik, nevodra: beside Detatar; nobodra: beside Nevodra; sizes " + "/".join(DETATAR_SIZES) + ")")
     args = ap.parse_args()
     if args.design:
         return run_design(args)

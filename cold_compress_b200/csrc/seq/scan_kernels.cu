@@ -333,8 +333,10 @@ __global__ void __launch_bounds__(J / (4 * NC) * 32, J >= 32 ? 2 : 4) delta_scan
     for (int e = 0; e < NC; ++e)
 #pragma unroll
         for (int c = 0; c < CH; ++c) st[e][c] = (n0 + c < D && j + e < a.V) ? S[(size_t)(n0 + c) * a.V + j + e] : 0.f;
-    for (int idx = tid; idx < 2 * buf_floats; idx += NTH) sm[idx] = 0.f;   // rows beyond D and padding stay zero
-    __syncthreads();
+    if (D != DL_PARTS * CH) {      // rows beyond D stay zero
+        for (int idx = tid; idx < 2 * buf_floats; idx += NTH) sm[idx] = 0.f;
+        __syncthreads();
+    }
     const float lam = expf(a.A_log[h]);
     auto at = [](int n) { return (n / CH) * RUN + (n % CH); };
     const bool vec = a.prepared && (D & 3) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.a_raw) & 15) == 0 && (a.ldqk & 3) == 0 &&
@@ -633,10 +635,19 @@ static int launch_delta_j(const CcSeqDeltaScan* a, cudaStream_t st) {
     return cuda_check("delta_scan_kernel");
 }
 
-template <int CH, int NC, int TB>
+// 32 value columns per CTA when that fills the GPU, else 16: half as many warps then share an SM's shared-memory reads
+// (measured for 4096 tokens of 8 / 16 / 32 heads x 128 x 128, decay per head: 32 columns 1.20 / 1.22 / 1.26 ms, 16 columns
+// 0.93 / 0.94 / 1.32 ms, 8 columns 0.97 / 1.03 / 1.39 ms)
+template <int CH, int NC, int TB, bool HD>
+static int launch_delta_hd(const CcSeqDeltaScan* a, cudaStream_t st) {
+    if (a->H * ((a->V + SCAN_J - 1) / SCAN_J) >= 96) return launch_delta_j<CH, NC, TB, SCAN_J, HD>(a, st);
+    return launch_delta_j<CH, NC, TB, SCAN_J / 2, HD>(a, st);
+}
+
+template <int CH, int NC>
 static int launch_delta(const CcSeqDeltaScan* a, cudaStream_t st) {
-    if (a->head_decay) return launch_delta_j<CH, NC, TB, SCAN_J, true>(a, st);
-    return launch_delta_j<CH, NC, TB, SCAN_J, false>(a, st);
+    if (a->T == 1) return a->head_decay ? launch_delta_hd<CH, NC, 1, true>(a, st) : launch_delta_hd<CH, NC, 1, false>(a, st);
+    return a->head_decay ? launch_delta_hd<CH, NC, 16, true>(a, st) : launch_delta_hd<CH, NC, 16, false>(a, st);
 }
 
 }  // namespace ccn
@@ -712,9 +723,9 @@ int cc_seq_delta_scan(const CcSeqDeltaScan* a, void* stream) {
     if (a->D > 256) return fail(CC_SEQ_ERR_UNSUPPORTED_SHAPE, "delta_scan: key heads wider than 256");
     cudaStream_t st = (cudaStream_t)stream;
     // rows per lane (8 lanes share a column's rows) x columns per lane
-    if (a->D <= 64) return launch_delta<8, DL_NC, 16>(a, st);
-    if (a->D <= 128) return launch_delta<16, DL_NC, 16>(a, st);
-    return launch_delta<32, DL_NC, 16>(a, st);
+    if (a->D <= 64) return launch_delta<8, DL_NC>(a, st);
+    if (a->D <= 128) return launch_delta<16, DL_NC>(a, st);
+    return launch_delta<32, DL_NC>(a, st);
 }
 
 int cc_seq_gated_rms_groups(const float* y, const float* gate, int64_t ldg, int32_t gate_act, int32_t gate_first,
