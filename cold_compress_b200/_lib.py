@@ -189,11 +189,20 @@ GEMV_MAX_JOBS = 6
 
 
 class CcSeqGemvJob(C.Structure):
-    _fields_ = [("x", _vp), ("W", _vp), ("out", _vp)] + [(n, _i32) for n in ("x_dtype", "kind", "off_gate", "off_up", "N", "K")]
+    _fields_ = [("x", _vp), ("W", _vp), ("out", _vp)] + [(n, _i32) for n in ("x_dtype", "kind", "off_gate", "off_up", "N", "K")] + [
+        ("conv_w", _vp), ("tail", _vp)] + [(n, _i32) for n in ("conv_rows", "taps", "conv_act")]
+
+
+GEMV_PRE_NONE, GEMV_PRE_OUTPUT_NORM, GEMV_PRE_GATED_HEADS = range(3)
+
+
+class CcSeqGemvPre(C.Structure):
+    _fields_ = [(n, _i32) for n in ("kind", "top", "w_len", "gate_act")] + [(n, _vp) for n in ("x", "y", "wts", "w", "gate", "x_out")] + [
+        ("eps", _f32), ("gain_offset", _f32)]
 
 
 class CcSeqGemvMulti(C.Structure):
-    _fields_ = [("job", CcSeqGemvJob * GEMV_MAX_JOBS), ("n_jobs", _i32), ("w_dtype", _i32)]
+    _fields_ = [("job", CcSeqGemvJob * GEMV_MAX_JOBS), ("n_jobs", _i32), ("w_dtype", _i32), ("pre", CcSeqGemvPre)]
 
 
 class CcSeqLatentPrep(C.Structure):
@@ -312,7 +321,10 @@ class CcSeqPostNorm(C.Structure):
                 ("next_offset", _f32), ("T", _i32), ("E", _i32)]
 
 
-SEQ_EXPORTS.update({"cc_seq_post_norm": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp])})
+SEQ_EXPORTS.update({
+    "cc_seq_post_norm": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp]),
+    "cc_seq_post_norm_route": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp, _vp, _i32, _i32, _vp, _vp, _vp]),
+})
 
 _seq_lib = None
 

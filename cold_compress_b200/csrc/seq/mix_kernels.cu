@@ -58,6 +58,14 @@ __device__ __forceinline__ void load8(const bf16* p, float* o) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) o[i] = __bfloat162float(e[i]);
 }
+__device__ __forceinline__ void st4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void st4(bf16* p, const float* v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+}
 // One weight row against one input row, by a warp: eight elements per lane and load when both rows allow it.
 template <typename WT, typename XT>
 __device__ __forceinline__ float warp_dot(const WT* __restrict__ w, const XT* __restrict__ x, int K, int lane) {
@@ -174,6 +182,24 @@ __global__ void gated_unit_kernel(const float* __restrict__ in, int64_t ld, int 
         float v = unit_act(row[off_gate + f], kind);
         if (off_up >= 0) v *= row[off_up + f];
         stf(out, (size_t)t * F + f, v);
+    }
+}
+
+// The same with four columns per thread (16-byte loads, one store), for rows whose offsets and stride allow it.
+template <typename ST>
+__global__ void gated_unit4_kernel(const float* __restrict__ in, int64_t ld, int off_gate, int off_up, ST* __restrict__ out,
+                                   int T, int F, int kind) {
+    const int f = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (f >= F) return;
+    for (int t = blockIdx.y; t < T; t += gridDim.y) {
+        const float* row = in + (size_t)t * ld + f;
+        const float4 a = *reinterpret_cast<const float4*>(row + off_gate);
+        float v[4] = {unit_act(a.x, kind), unit_act(a.y, kind), unit_act(a.z, kind), unit_act(a.w, kind)};
+        if (off_up >= 0) {
+            const float4 u = *reinterpret_cast<const float4*>(row + off_up);
+            v[0] *= u.x; v[1] *= u.y; v[2] *= u.z; v[3] *= u.w;
+        }
+        st4(out + (size_t)t * F + f, v);
     }
 }
 
@@ -843,16 +869,90 @@ static int dispatch_latent_decode(const CcSeqLatentDecode* a, cudaStream_t st) {
 __device__ __forceinline__ float round_to(float v, const float*) { return v; }
 __device__ __forceinline__ float round_to(float v, const bf16*) { return __bfloat162float(__float2bfloat16_rn(v)); }
 
+// The launch's shared input row, formed by every CTA (see CcSeqGemvPre): xs[K], rounded to the weights' type.
+template <typename WT, int VEC>
+__device__ __forceinline__ void gemv_output_norm_row(const CcSeqGemvPre& p, float* xs, int K, bool first_cta, float* red, const WT* W) {
+    struct alignas(VEC == 4 ? 16 : 4) Pack { float v[VEC]; };
+    auto ld = [](const float* q) { return *reinterpret_cast<const Pack*>(q); };
+    const int tid = threadIdx.x;
+    float ss = 0.f;
+    for (int k = tid * VEC; k < K; k += 256 * VEC) {
+        Pack r;
+        if (p.top == 0) {
+            r = ld(p.y + k);
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) r.v[i] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < p.top; ++j) {
+                const Pack y = ld(p.y + (size_t)j * K + k);
+                const float w = p.wts[j];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) r.v[i] = fmaf(w, y.v[i], r.v[i]);
+            }
+        }
+        *reinterpret_cast<Pack*>(xs + k) = r;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(r.v[i], r.v[i], ss);
+    }
+    const float rinv = 1.0f / sqrtf(block_sum(ss, red) / (float)K + p.eps);
+    for (int k = tid * VEC; k < K; k += 256 * VEC) {
+        const Pack x = ld(p.x + k), w = ld(p.w + k), r = ld(xs + k);
+        Pack s;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s.v[i] = x.v[i] + r.v[i] * rinv * (w.v[i] + p.gain_offset);
+        if (first_cta) *reinterpret_cast<Pack*>(p.x_out + k) = s;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s.v[i] = round_to(s.v[i], W);
+        *reinterpret_cast<Pack*>(xs + k) = s;
+    }
+}
+
 template <typename WT>
+__device__ __forceinline__ void gemv_gated_heads_row(const CcSeqGemvPre& p, float* xs, int K, const WT* W) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, V = p.w_len;
+    for (int h = warp; h < K / V; h += 8) {
+        const float* y = p.y + (size_t)h * V;
+        const float* gate = p.gate + (size_t)h * V;
+        float ss = 0.f;
+        for (int e = lane; e < V; e += 32) ss = fmaf(y[e], y[e], ss);
+        const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)V + p.eps);
+        for (int e = lane; e < V; e += 32) xs[h * V + e] = round_to(y[e] * rinv * p.w[e] * unit_act(gate[e], p.gate_act), W);
+    }
+}
+
+template <typename WT, int PRE>
 __global__ void __launch_bounds__(256) gemv_multi_kernel(const CcSeqGemvMulti g) {
     extern __shared__ float4 smg4[];
     float* xs = reinterpret_cast<float*>(smg4);
+    __shared__ float red[32];
     int j = 0, first = 0;
     while (j + 1 < g.n_jobs && (int)blockIdx.x >= first + (g.job[j].N + 7) / 8) { first += (g.job[j].N + 7) / 8; ++j; }
     const CcSeqGemvJob& jb = g.job[j];
     const int K = jb.K, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const WT* W = (const WT*)jb.W;
-    if (jb.kind != CC_ACT_NONE || jb.off_up >= 0) {
+    const int n = ((int)blockIdx.x - first) * 8 + warp;
+    const WT* w = W + (size_t)min(n, jb.N - 1) * K;
+    constexpr int VEC = 16 / (int)sizeof(WT), AHEAD = 4;
+    const bool vec = K % VEC == 0;
+    // with a shared row to form, the row's first weights are requested before it
+    uint4 ahead[PRE != CC_GEMV_PRE_NONE ? AHEAD : 1];
+    if constexpr (PRE != CC_GEMV_PRE_NONE) {
+        const uint4* w16 = reinterpret_cast<const uint4*>(w);
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a) ahead[a] = vec && lane + 32 * a < K / VEC ? __ldg(w16 + lane + 32 * a) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    bool shared_row = false;
+    if constexpr (PRE != CC_GEMV_PRE_NONE) shared_row = jb.x == nullptr;
+    if (shared_row) {
+        if constexpr (PRE == CC_GEMV_PRE_OUTPUT_NORM) {
+            const uintptr_t all = (uintptr_t)g.pre.x | (uintptr_t)g.pre.y | (uintptr_t)g.pre.w | (uintptr_t)g.pre.x_out;
+            if (K % 4 == 0 && (all & 15) == 0) gemv_output_norm_row<WT, 4>(g.pre, xs, K, blockIdx.x == 0, red, W);
+            else gemv_output_norm_row<WT, 1>(g.pre, xs, K, blockIdx.x == 0, red, W);
+        } else if constexpr (PRE == CC_GEMV_PRE_GATED_HEADS) {
+            gemv_gated_heads_row<WT>(g.pre, xs, K, W);
+        }
+    } else if (jb.kind != CC_ACT_NONE || jb.off_up >= 0) {
         const float* src = (const float*)jb.x;
         for (int k = tid; k < K; k += 256) {
             float v = unit_act(src[jb.off_gate + k], jb.kind);
@@ -865,33 +965,49 @@ __global__ void __launch_bounds__(256) gemv_multi_kernel(const CcSeqGemvMulti g)
         for (int k = tid; k < K; k += 256) xs[k] = __bfloat162float(((const bf16*)jb.x)[k]);
     }
     __syncthreads();
-    const int n = ((int)blockIdx.x - first) * 8 + warp;
     if (n >= jb.N) return;
-    const WT* w = W + (size_t)n * K;
-    constexpr int VEC = 16 / (int)sizeof(WT);
     float acc = 0.f;
-    if (K % VEC == 0) {
+    auto dot16 = [&](const uint4& u, int i) {
+        const WT* e = reinterpret_cast<const WT*>(&u);
+        const float4* x4 = reinterpret_cast<const float4*>(xs + i * VEC);
+#pragma unroll
+        for (int q = 0; q < VEC / 4; ++q) {
+            const float4 xv = x4[q];
+            acc = fmaf(ldf(e, 4 * q + 0), xv.x, acc);
+            acc = fmaf(ldf(e, 4 * q + 1), xv.y, acc);
+            acc = fmaf(ldf(e, 4 * q + 2), xv.z, acc);
+            acc = fmaf(ldf(e, 4 * q + 3), xv.w, acc);
+        }
+    };
+    if (vec) {
         const uint4* w16 = reinterpret_cast<const uint4*>(w);
         const int nv = K / VEC;
-#pragma unroll 4
-        for (int i = lane; i < nv; i += 32) {
-            const uint4 u = __ldg(w16 + i);
-            const WT* e = reinterpret_cast<const WT*>(&u);
-            const float4* x4 = reinterpret_cast<const float4*>(xs + i * VEC);
+        int i = lane;
+        if constexpr (PRE != CC_GEMV_PRE_NONE) {
 #pragma unroll
-            for (int q = 0; q < VEC / 4; ++q) {
-                const float4 xv = x4[q];
-                acc = fmaf(ldf(e, 4 * q + 0), xv.x, acc);
-                acc = fmaf(ldf(e, 4 * q + 1), xv.y, acc);
-                acc = fmaf(ldf(e, 4 * q + 2), xv.z, acc);
-                acc = fmaf(ldf(e, 4 * q + 3), xv.w, acc);
-            }
+            for (int a = 0; a < AHEAD; ++a, i += 32)
+                if (i < nv) dot16(ahead[a], i);
         }
+#pragma unroll 4
+        for (; i < nv; i += 32) dot16(__ldg(w16 + i), i);
     } else {
         for (int k = lane; k < K; k += 32) acc = fmaf(ldf(w, k), xs[k], acc);
     }
     acc = warp_sum(acc);
-    if (lane == 0) ((float*)jb.out)[n] = acc;
+    if (lane != 0) return;
+    if (n < jb.conv_rows) {      // this row is a channel: its past inputs, then the tail moves on
+        const int C = jb.conv_rows, taps = jb.taps;
+        const float* cw = jb.conv_w + (size_t)n * taps;
+        float c = 0.f;
+        for (int t = 0; t < taps - 1; ++t) {
+            const float u = jb.tail[(size_t)t * C + n];
+            c = fmaf(cw[t], u, c);
+            if (t > 0) jb.tail[(size_t)(t - 1) * C + n] = u;
+        }
+        if (taps > 1) jb.tail[(size_t)(taps - 2) * C + n] = acc;
+        acc = unit_act(fmaf(cw[taps - 1], acc, c), jb.conv_act);
+    }
+    ((float*)jb.out)[n] = acc;
 }
 
 template <int TB, int CH>
@@ -984,6 +1100,14 @@ int cc_seq_gated_unit(const float* in, int64_t ld, int32_t off_gate, int32_t off
     if (!in || !out || T < 1 || F < 1 || kind < CC_ACT_NONE || kind > CC_ACT_LAST)
         return fail(CC_SEQ_ERR_INVALID_ARG, "gated_unit: bad argument");
     cudaStream_t st = (cudaStream_t)stream;
+    if (F % 4 == 0 && ld % 4 == 0 && off_gate % 4 == 0 && (off_up < 0 || off_up % 4 == 0) && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+        const int threads = F / 4 >= 256 ? 256 : (F / 4 + 31) / 32 * 32;
+        const dim3 nb4((F / 4 + threads - 1) / threads, T < 4096 ? T : 4096);
+#define CALL(ST) gated_unit4_kernel<ST><<<nb4, threads, 0, st>>>(in, ld, off_gate, off_up, (ST*)out, T, F, kind)
+        CCM_ST(out_dtype, CALL);
+#undef CALL
+        return cuda_check("gated_unit4_kernel");
+    }
     const dim3 nb((F + 255) / 256, T < 4096 ? T : 4096);
 #define CALL(ST) gated_unit_kernel<ST><<<nb, 256, 0, st>>>(in, ld, off_gate, off_up, (ST*)out, T, F, kind)
     CCM_ST(out_dtype, CALL);
@@ -1144,21 +1268,34 @@ int cc_seq_latent_decode(const CcSeqLatentDecode* a, void* stream) {
 
 int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream) {
     if (!g || g->n_jobs < 1 || g->n_jobs > CC_GEMV_MAX_JOBS) return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad job count");
+    const CcSeqGemvPre& p = g->pre;
     int blocks = 0, kmax = 0;
     for (int j = 0; j < g->n_jobs; ++j) {
         const CcSeqGemvJob& b = g->job[j];
-        if (!b.x || !b.W || !b.out || b.N < 1 || b.K < 1 || b.kind < CC_ACT_NONE || b.kind > CC_ACT_LAST ||
+        if (!b.W || !b.out || b.N < 1 || b.K < 1 || b.kind < CC_ACT_NONE || b.kind > CC_ACT_LAST ||
             ((b.kind != CC_ACT_NONE || b.off_up >= 0) && b.x_dtype != CC_DT_F32))
             return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad job");
+        if (b.conv_rows < 0 || b.conv_rows > b.N || (b.conv_rows > 0 && (!b.conv_w || b.taps < 1 || (b.taps > 1 && !b.tail) ||
+                                                                         b.conv_act < CC_ACT_NONE || b.conv_act > CC_ACT_LAST)))
+            return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad convolution");
+        if (!b.x) {
+            const bool ok = p.kind == CC_GEMV_PRE_OUTPUT_NORM ? p.x && p.y && p.w && p.x_out && p.x_out != p.x && p.top >= 0 && (p.top == 0 || p.wts) :
+                            p.kind == CC_GEMV_PRE_GATED_HEADS ? p.y && p.w && p.gate && p.w_len >= 1 && b.K % p.w_len == 0 &&
+                                                                p.gate_act >= CC_ACT_NONE && p.gate_act <= CC_ACT_LAST : false;
+            // CTA 0 belongs to job 0: it is the one that hands the summed row on
+            if (!ok || b.kind != CC_ACT_NONE || b.off_up >= 0 || g->job[0].x || b.K != g->job[0].K)
+                return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad shared input row");
+        }
         blocks += (b.N + 7) / 8;
         kmax = b.K > kmax ? b.K : kmax;
     }
+    if (p.kind < CC_GEMV_PRE_NONE || p.kind > CC_GEMV_PRE_GATED_HEADS) return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: unknown shared input row");
     const size_t smem = sizeof(float) * (size_t)((kmax + 3) & ~3);
     if (smem > 200 * 1024) return fail(CC_SEQ_ERR_UNSUPPORTED_SHAPE, "gemv_multi: input longer than 51200");
     cudaStream_t st = (cudaStream_t)stream;
-#define CALL(ST)                                                                                                   \
+#define CALL1(ST, PRE)                                                                                             \
     {                                                                                                              \
-        auto kern = gemv_multi_kernel<ST>;                                                                         \
+        auto kern = gemv_multi_kernel<ST, PRE>;                                                                    \
         static size_t configured = 48 * 1024;                                                                      \
         if (smem > configured) {                                                                                   \
             configured = smem;                                                                                     \
@@ -1167,8 +1304,15 @@ int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream) {
         }                                                                                                          \
         kern<<<blocks, 256, smem, st>>>(*g);                                                                       \
     }
+#define CALL(ST)                                                                        \
+    {                                                                                   \
+        if (p.kind == CC_GEMV_PRE_OUTPUT_NORM) CALL1(ST, CC_GEMV_PRE_OUTPUT_NORM)       \
+        else if (p.kind == CC_GEMV_PRE_GATED_HEADS) CALL1(ST, CC_GEMV_PRE_GATED_HEADS)  \
+        else CALL1(ST, CC_GEMV_PRE_NONE)                                                \
+    }
     CCM_ST(g->w_dtype, CALL);
 #undef CALL
+#undef CALL1
     return cuda_check("gemv_multi_kernel");
 }
 

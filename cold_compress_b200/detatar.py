@@ -434,14 +434,18 @@ class RoutedExperts(nn.Module):
         if rows:
             xs = torch.empty(rows, E, dtype=dt, device=dev)
             seq_ops.gather_rows(h_act, perm, xs, rows)
-            lo = 0
+            up = torch.empty(rows, self.w_gu.shape[1], dtype=torch.float32, device=dev)
+            act = torch.empty(rows, F, dtype=dt, device=dev)
+            spans, lo = [], 0
             for e, cnt in enumerate(sizes):
                 if cnt:
-                    gu = _mm(xs[lo:lo + cnt], self.w_gu[e])
-                    act = torch.empty(cnt, F, dtype=dt, device=dev)
-                    seq_ops.gated_unit(gu, 0, F if self.gated else -1, act, self.act)
-                    _mm(act, self.w_d[e], out=y[lo:lo + cnt])
+                    spans.append((e, lo, lo + cnt))
                     lo += cnt
+            for e, lo, hi in spans:
+                _mm(xs[lo:hi], self.w_gu[e], out=up[lo:hi])
+            seq_ops.gated_unit(up, 0, F if self.gated else -1, act, self.act)
+            for e, lo, hi in spans:
+                _mm(act[lo:hi], self.w_d[e], out=y[lo:hi])
         return slot, y
 
 

@@ -126,6 +126,13 @@ class KeyValueAttention(nn.Module):
         cache.sequence_step(q, k, v, ip, y, window=self.window, scale=self.scale)
         return y.view(T, self.nq)
 
+    def input_conv(self, store):
+        return None
+
+    def close_one_token(self, hp: Tensor, ip: Tensor, cache, out: Tensor):
+        """One token, from the input product's row to the mixer's output."""
+        seq_ops.gemv_multi([(self.core(hp, ip, cache, True), self.w_o, out)])
+
 
 class DeltaMixer(nn.Module):
     """`tefovik.GatedDeltaRule` as a mixer of its own: one decay per head, a full-rank output gate, and the projection
@@ -142,6 +149,19 @@ class DeltaMixer(nn.Module):
 
     def core(self, hp: Tensor, ip: Tensor, state, one_token: bool) -> Tensor:
         return self.rule.core(hp, 0, ip, state, one_token)
+
+    def input_conv(self, state):
+        """One token: the short convolution runs inside the input product's launch (a channel is a row of it)."""
+        return self.rule.conv.weight, state.vectors, self.rule.conv.act
+
+    def close_one_token(self, hp: Tensor, ip: Tensor, state, out: Tensor):
+        """One token, from the input product's row (its convolution applied) to the mixer's output: the recurrence, then the
+        output product, which forms the normed and gated heads itself."""
+        r = self.rule
+        a = r.conv_width + r.heads
+        g = a + r.a_rows
+        o = r.scan(hp[:, :r.conv_width], hp[:, r.conv_width:a], hp[:, a:g], state)
+        seq_ops.gemv_multi([(None, r.w_o, out)], pre=seq_ops.gated_heads_row(o, r.norm_w, hp[:, g:g + r.g_rows], r.gate_act, r.eps))
 
 
 # --------------------------------------------------------------------------------------------- a layer
@@ -188,10 +208,45 @@ class NobodraBlock(nn.Module):
         if self.mlp is not None:
             self.norm2(x, self.fed(x_act, one_token), side)
 
+    def step_one_token(self, x: Tensor, copy: Optional[Tensor], ip: Tensor, pending: Optional[tuple]):
+        """The same layer for one token; `copy` is scratch for the stream in the compute dtype (None in fp32).  `pending` is
+        the sublayer result of the layer before with its norm: the input product's launch adds it to the stream (into a new
+        buffer: its CTAs read the old row).  Then the mixer, the norm + sum + router in one launch, and the experts, whose
+        weighted sum is this layer's pending result.  Returns (stream, pending)."""
+        hp, mixed, conv = _out(self.mixer.w_in), _out(self.mixer.w_o), self.mixer.input_conv(self.store)
+        if pending is None:
+            seq_ops.gemv_multi([(x, self.mixer.w_in, hp)], conv=conv)
+        else:
+            result, norm = pending
+            total = torch.empty_like(x)
+            pre = seq_ops.output_norm_row(x, result["y"], norm.weight, norm.eps, norm.gain_offset, total, wts=result.get("wts"))
+            seq_ops.gemv_multi([(None, self.mixer.w_in, hp)], pre=pre, conv=conv)
+            x = total
+        self.mixer.close_one_token(hp, ip, self.store, mixed)
+        f = self.mlp
+        if f is None:
+            return x, (dict(y=mixed), self.norm1)
+        if self.routes_with_norm():
+            ids = torch.empty(1, f.top, dtype=torch.int32, device=x.device)
+            wts = torch.empty(1, f.top, dtype=torch.float32, device=x.device)
+            seq_ops.post_norm_route(x, mixed, self.norm1.weight, self.norm1.eps, self.norm1.gain_offset, self.w_router, f.correction,
+                                    ids, wts, x_act=copy)
+        else:
+            self.norm1(x, dict(y=mixed), copy)
+            ids, wts = f.route(_product(x if copy is None else copy, self.w_router, True), 0)
+        _, y = f.expert_rows(ids, x if copy is None else copy)
+        return x, (dict(y=y, wts=wts), self.norm2)
+
+    # one CTA reads the whole router in the fused launch: beyond this a launch of its own, spread over the GPU, is faster
+    ROUTER_BYTES = 1 << 19
+
+    def routes_with_norm(self) -> bool:
+        return self.w_router.numel() * self.w_router.element_size() <= self.ROUTER_BYTES
+
     def kernels_per_token(self):
-        # input product, core (q/k/v rows + attention, or convolution + scan + gated norm), output product, norm + sum;
-        # router product, choice, experts up and down, sum + norm
-        return 3 + (2 if self.kind == "attention" else 3) + (5 if self.mlp is not None else 0)
+        # input product (with the norm + sum of the layer before and the convolution), q/k/v rows + attention or the scan,
+        # output product; norm + sum + router, experts up and down
+        return (4 if self.kind == "attention" else 3) + (0 if self.mlp is None else 3 if self.routes_with_norm() else 5)
 
 
 # --------------------------------------------------------------------------------------------- the model
@@ -287,6 +342,8 @@ class NobodraTransformer(nn.Module):
         x = torch.empty(T, E, dtype=torch.float32, device=dev)
         x_act = x if dt == torch.float32 else torch.empty(T, E, dtype=dt, device=dev)
         seq_ops.embed_rows(tokens, self.tok_embeddings, x, 1.0)
+        if one and collect is None and len(self.layers):
+            return self._step_one_token(x, None if x_act is x else x_act, ip)
         if x_act is not x:
             seq_ops.gated_unit(x, 0, -1, x_act, _lib.ACT_NONE)
         for layer in self.layers:
@@ -300,9 +357,20 @@ class NobodraTransformer(nn.Module):
         seq_ops.sum_norm(self.norm.weight, self.norm.eps, x=x, center=False, gain_offset=self.norm.gain_offset, rows=rows, out_act=xs_act)
         return _product(xs_act, self.output, one).view(1, rows.numel(), -1)
 
+    def _step_one_token(self, x: Tensor, copy: Optional[Tensor], ip: Tensor) -> Tensor:
+        pending = None
+        for layer in self.layers:
+            x, pending = layer.step_one_token(x, copy, ip, pending)
+        result, norm = pending
+        xs_act = torch.empty_like(x) if copy is None else copy
+        norm(x, result, xs_act, then=self.norm)
+        logits = _out(self.output)
+        seq_ops.gemv_multi([(xs_act, self.output, logits)])
+        return logits.view(1, 1, -1)
+
     def kernels_per_token(self) -> int:
         """Launches of this package's kernels in one decode step (fused_decode)."""
-        return 4 + sum(l.kernels_per_token() for l in self.layers)   # embedding row, its copy; last norm, head
+        return 3 + sum(l.kernels_per_token() for l in self.layers)   # embedding row; last sum + both norms, head
 
     # ---- weights --------------------------------------------------------------------------------
     def load_tensors(self, tensors: Dict[str, Tensor]):

@@ -444,9 +444,11 @@ def latent_decode(q, k_new, k_cache, pos, mask, cache_cts, input_pos, y, scale, 
     _lib.check_seq(_lib.load_seq().cc_seq_latent_decode(C.byref(a), _stream()), "cc_seq_latent_decode")
 
 
-def gemv_multi(jobs):
+def gemv_multi(jobs, pre=None, conv=None):
     """Up to six one-token products in one launch.  jobs: (x, w, out) or (src, w, out, kind, off_gate, off_up) where the
-    input is built from the fp32 row `src` as act(src[off_gate + k]) * src[off_up + k]; out fp32 [1, N]."""
+    input is built from the fp32 row `src` as act(src[off_gate + k]) * src[off_up + k]; out fp32 [1, N].  x = None: the
+    launch's shared row `pre` (output_norm_row or gated_heads_row), which every CTA forms for itself.  conv = (table
+    [C, taps], tail [taps - 1, C], act): the first C rows of job 0 pass that short convolution, whose tail moves on."""
     g = _lib.CcSeqGemvMulti()
     g.n_jobs = len(jobs)
     assert 1 <= len(jobs) <= _lib.GEMV_MAX_JOBS
@@ -457,11 +459,45 @@ def gemv_multi(jobs):
         _need(("x", x, None), ("w", w, jobs[0][1].dtype), ("out", out, torch.float32))
         N, K = w.shape
         built = kind != _lib.ACT_NONE or off_up >= 0
-        assert out.numel() == N and (x.numel() >= max(off_gate, off_up) + K if built else x.numel() == K)
+        assert out.numel() == N and (pre.length == K if x is None else x.numel() >= max(off_gate, off_up) + K if built else x.numel() == K)
         b = g.job[j]
         b.x, b.W, b.out = _p(x), _p(w), _p(out)
-        b.x_dtype, b.kind, b.off_gate, b.off_up, b.N, b.K = _dt(x), int(kind), int(off_gate), int(off_up), N, K
+        b.x_dtype, b.kind, b.off_gate, b.off_up, b.N, b.K = _dt(x) if x is not None else _lib.DT_F32, int(kind), int(off_gate), int(off_up), N, K
+    if pre is not None:
+        g.pre = pre
+    if conv is not None:
+        table, tail, act = conv
+        _need(("table", table, torch.float32), ("tail", tail, torch.float32))
+        b = g.job[0]
+        b.conv_rows, b.taps = table.shape
+        assert b.conv_rows <= b.N and tail.shape == (b.taps - 1, b.conv_rows)
+        b.conv_w, b.tail, b.conv_act = _p(table), (_p(tail) if b.taps > 1 else None), int(act)
     _lib.check_seq(_lib.load_seq().cc_seq_gemv_multi(C.byref(g), _stream()), "cc_seq_gemv_multi")
+
+
+def output_norm_row(x, y, w, eps, gain_offset, x_out, wts=None):
+    """Shared input row for gemv_multi: x + rms_norm(r) * (w + gain_offset) for one token (r = y [1, E], or the sum of
+    wts[k] * y[k] over the rows of y), also written to x_out."""
+    _need(("x", x, torch.float32), ("y", y, torch.float32), ("w", w, torch.float32), ("x_out", x_out, torch.float32), ("wts", wts, torch.float32))
+    E = w.numel()
+    assert x.numel() == E and x_out.numel() == E and x_out.data_ptr() != x.data_ptr() and y.numel() >= E * (1 if wts is None else wts.numel())
+    p = _lib.CcSeqGemvPre()
+    p.kind, p.x, p.y, p.w, p.x_out, p.eps, p.gain_offset = _lib.GEMV_PRE_OUTPUT_NORM, _p(x), _p(y), _p(w), _p(x_out), float(eps), float(gain_offset)
+    p.wts, p.top = _p(wts), 0 if wts is None else wts.numel()
+    p.length = E
+    return p
+
+
+def gated_heads_row(y, w, gate, act, eps):
+    """Shared input row for gemv_multi: every part of len(w) entries of y [1, K] RMS-normed times w, times act(gate [1, K])."""
+    _need(("y", y, torch.float32), ("w", w, torch.float32))
+    p = _lib.CcSeqGemvPre()
+    K = y.numel()
+    gp, _ = _cols(_f32("gate", gate))
+    assert gate.numel() == K and K % w.numel() == 0
+    p.kind, p.y, p.w, p.gate, p.gate_act, p.w_len, p.eps = _lib.GEMV_PRE_GATED_HEADS, _p(y), _p(w), gp, int(act), w.numel(), float(eps)
+    p.length = K
+    return p
 
 
 # ------------------------------------------------------------------------------------------------------------------
@@ -649,13 +685,9 @@ def poly_norm(src, coef, out, eps):
 # ------------------------------------------------------------------------------------------------------------------
 # Fifth part of the C ABI (csrc/seq/post_kernels.cu): sublayer outputs that are normed before they join the stream.
 
-def post_norm(x, y, w, eps, gain_offset=0.0, wts=None, slot=None, x_out=None, x_act=None, next_w=None, next_eps=0.0,
-              next_offset=0.0):
-    """x (fp32 [T, E]) + rms_norm(r) * (w + gain_offset) -> x_out (default: x in place), with r the row of y [T, E] or,
-    with wts [T, top], the weighted sum of the rows slot[t, k] (default t * top + k) of y [*, E].  x_act: the sum in the
-    compute dtype, or the RMS norm of it with gain next_w + next_offset."""
+def _post_norm_args(x, y, w, eps, gain_offset, wts=None, slot=None, x_out=None, x_act=None):
     _need(("x", x, torch.float32), ("w", w, torch.float32), ("wts", wts, torch.float32), ("slot", slot, torch.int32),
-          ("x_out", x_out, torch.float32), ("x_act", x_act, None), ("next_w", next_w, torch.float32))
+          ("x_out", x_out, torch.float32), ("x_act", x_act, None))
     a = _lib.CcSeqPostNorm()
     T, E = x.shape
     a.y, a.ldy = _cols(_f32("y", y))
@@ -663,6 +695,29 @@ def post_norm(x, y, w, eps, gain_offset=0.0, wts=None, slot=None, x_out=None, x_
     assert (y.shape[0] == T) if wts is None else (wts.shape[0] == T and a.ldy == E and (slot is not None or y.shape[0] >= wts.numel()))
     a.x, a.wts, a.slot, a.top = _p(x), _p(wts), _p(slot), 0 if wts is None else wts.shape[1]
     a.w, a.eps, a.gain_offset, a.x_out = _p(w), float(eps), float(gain_offset), _p(x_out)
-    a.x_act, a.act_dtype = _p(x_act), _dt(x_act) if x_act is not None else _lib.DT_F32
-    a.next_w, a.next_eps, a.next_offset, a.T, a.E = _p(next_w), float(next_eps), float(next_offset), T, E
+    a.x_act, a.act_dtype, a.T, a.E = _p(x_act), _dt(x_act) if x_act is not None else _lib.DT_F32, T, E
+    return a
+
+
+def post_norm(x, y, w, eps, gain_offset=0.0, wts=None, slot=None, x_out=None, x_act=None, next_w=None, next_eps=0.0,
+              next_offset=0.0):
+    """x (fp32 [T, E]) + rms_norm(r) * (w + gain_offset) -> x_out (default: x in place), with r the row of y [T, E] or,
+    with wts [T, top], the weighted sum of the rows slot[t, k] (default t * top + k) of y [*, E].  x_act: the sum in the
+    compute dtype, or the RMS norm of it with gain next_w + next_offset."""
+    _need(("next_w", next_w, torch.float32))
+    a = _post_norm_args(x, y, w, eps, gain_offset, wts, slot, x_out, x_act)
+    a.next_w, a.next_eps, a.next_offset = _p(next_w), float(next_eps), float(next_offset)
     _lib.check_seq(_lib.load_seq().cc_seq_post_norm(C.byref(a), _stream()), "cc_seq_post_norm")
+
+
+def post_norm_route(x, y, w, eps, gain_offset, router, bias, ids, wts, x_act=None, x_out=None):
+    """post_norm of a few tokens' rows y [T, E], then the router that reads the sum: the ids.shape[1] largest of
+    `router[:len(bias)] @ s + bias` per token and the softmax over them.  router [>= n, E] in the compute dtype (x_act's)."""
+    _need(("router", router, None), ("bias", bias, torch.float32), ("ids", ids, torch.int32), ("route_wts", wts, torch.float32))
+    a = _post_norm_args(x, y, w, eps, gain_offset, x_out=x_out, x_act=x_act)
+    n = bias.numel()
+    assert router.shape[0] >= n and router.shape[1] == a.E and ids.shape == wts.shape and ids.shape[0] == a.T
+    assert x_act is None or router.dtype == x_act.dtype
+    a.act_dtype = _dt(router)
+    _lib.check_seq(_lib.load_seq().cc_seq_post_norm_route(C.byref(a), _p(router), _p(bias), n, ids.shape[1], _p(ids), _p(wts), _stream()),
+                   "cc_seq_post_norm_route")

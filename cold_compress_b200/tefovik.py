@@ -269,16 +269,22 @@ class GatedDeltaRule(nn.Module):
 
     def core(self, hp: Tensor, off: int, ip: Tensor, state, one_token: bool) -> Tensor:
         T, dev, dt = hp.shape[0], hp.device, self.w_o.dtype
-        H, G, D, V = self.heads, self.kv_heads, self.head_dim, self.v_dim
+        H, V = self.heads, self.v_dim
         ob = off + self.conv_width
         c = self.conv(hp[:, off:off + self.conv_width], state.vectors)
         a_raw, g_raw = self._second_products(hp, ob + H, ob + H + self.a_rows, one_token)
-        o = torch.empty(T, H * V, dtype=torch.float32, device=dev)
-        seq_ops.delta_scan(c[:, :G * D], c[:, G * D:2 * G * D], c[:, 2 * G * D:], hp[:, ob:ob + H], a_raw, self.dt_bias, self.A_log,
-                           state.matrix, o, H, G, D, V, D ** -0.5, self.unit_eps)
+        o = self.scan(c, hp[:, ob:ob + H], a_raw, state)
         on = torch.empty(T, H * V, dtype=dt, device=dev)
         seq_ops.gated_rms_groups(o, g_raw, self.gate_act, False, self.norm_w, on, H, self.eps)
         return on
+
+    def scan(self, c: Tensor, beta_raw: Tensor, a_raw: Tensor, state) -> Tensor:
+        """The recurrence over rows c = [q | k | v] that have passed their convolution -> fp32 [T, heads * v_dim]."""
+        H, G, D, V = self.heads, self.kv_heads, self.head_dim, self.v_dim
+        o = torch.empty(c.shape[0], H * V, dtype=torch.float32, device=c.device)
+        seq_ops.delta_scan(c[:, :G * D], c[:, G * D:2 * G * D], c[:, 2 * G * D:], beta_raw, a_raw, self.dt_bias, self.A_log,
+                           state.matrix, o, H, G, D, V, D ** -0.5, self.unit_eps)
+        return o
 
 
 class ParallelMixer(nn.Module):

@@ -261,15 +261,33 @@ int cc_seq_latent_decode(const CcSeqLatentDecode* a, void* stream);
  * Several one-token products in one launch (job j: out_j fp32 [N] = W_j [N, K] xin_j).  xin_j = x (x_dtype: fp32 or
  * the weights' type), or, with kind != CC_ACT_NONE or off_up >= 0, built from the fp32 row x as
  * act(x[off_gate + k]) * x[off_up + k] (no second factor when off_up < 0): the input side of a gated unit.
+ * x == NULL: the input is the launch's shared row, which every CTA forms for itself from `pre`:
+ *   CC_GEMV_PRE_OUTPUT_NORM  s = x + r / sqrt(mean(r^2) + eps) * (w + gain_offset), r = y, or with top > 0 the sum of
+ *                            wts[k] * y[k * K ...] over k < top (what cc_seq_post_norm does for one row); s is also
+ *                            written to x_out (not x: other CTAs still read it)
+ *   CC_GEMV_PRE_GATED_HEADS  y[k] / (root mean square of its part of w_len entries) * w[k mod w_len] * act(gate[k])
+ * conv_rows > 0: rows n < conv_rows of the job then pass a causal convolution over time (a channel per row, the taps
+ * before the current one from `tail` fp32 [taps - 1, conv_rows], which is moved on) and the activation conv_act.
  */
 #define CC_GEMV_MAX_JOBS 6
+#define CC_GEMV_PRE_NONE         0
+#define CC_GEMV_PRE_OUTPUT_NORM  1
+#define CC_GEMV_PRE_GATED_HEADS  2
 typedef struct CcSeqGemvJob {
     const void* x;  const void* W;  void* out;
     int32_t x_dtype, kind, off_gate, off_up, N, K;
+    const float* conv_w;  float* tail;
+    int32_t conv_rows, taps, conv_act;
 } CcSeqGemvJob;
+typedef struct CcSeqGemvPre {
+    int32_t kind, top, w_len, gate_act;
+    const float* x;  const float* y;  const float* wts;  const float* w;  const float* gate;  float* x_out;
+    float eps, gain_offset;
+} CcSeqGemvPre;
 typedef struct CcSeqGemvMulti {
     CcSeqGemvJob job[CC_GEMV_MAX_JOBS];
     int32_t n_jobs, w_dtype;
+    CcSeqGemvPre pre;
 } CcSeqGemvMulti;
 int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream);
 
@@ -542,6 +560,15 @@ typedef struct CcSeqPostNorm {
     int32_t T, E;
 } CcSeqPostNorm;
 int cc_seq_post_norm(const CcSeqPostNorm* a, void* stream);
+
+/*
+ * The same sum for a step of few tokens, followed by the choice of the next feed-forward's experts, one CTA per token:
+ * logits = Wr [n, E] s + bias (s rounded to act_dtype, Wr in act_dtype), the `top` largest (the lower index on a tie)
+ * and the softmax over them: ids int32, wts fp32 [T, top].  The block's x_act (without next_w) is the experts' input;
+ * its wts / slot / top describe y as above.
+ */
+int cc_seq_post_norm_route(const CcSeqPostNorm* a, const void* Wr, const float* bias, int32_t n, int32_t top, int32_t* ids,
+                           float* wts, void* stream);
 
 #ifdef __cplusplus
 }

@@ -76,6 +76,107 @@ def test_output_norm_of_the_weighted_expert_rows(T, E, top):
         _close(x, x0.double() + R.rms_around_one(mixed, w.double(), 1e-5), 1e-6)
 
 
+# ----------------------------------------------------------------------------------------------- one-token launches
+
+@pytest.mark.parametrize("E,n,top", [(64, 6, 2), (51, 1, 1), (640, 40, 7), (2052, 9, 9), (4, 130, 3)])
+@pytest.mark.parametrize("T", [1, 3])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_output_norm_with_the_router_that_reads_the_sum(E, n, top, T, dtype):
+    ops = _ops()
+    g = torch.Generator().manual_seed(E + n)
+    x0, y, w = torch.randn(T, E, generator=g), torch.randn(T, E, generator=g), torch.randn(E, generator=g) * 0.5
+    router, bias = (torch.randn(n + 3, E, generator=g) * E ** -0.5 * 0.1).to(dtype), torch.randperm(n, generator=g).float()
+    want = x0.double() + R.rms_around_one(y.double(), w.double(), 1e-5)
+    x, act = x0.to(DEV), torch.empty(T, E, device=DEV, dtype=dtype)
+    ids, wts = torch.empty(T, top, dtype=torch.int32, device=DEV), torch.empty(T, top, device=DEV)
+    ops.post_norm_route(x, y.to(DEV), w.to(DEV), 1e-5, 1.0, router.to(DEV), bias.to(DEV), ids, wts, x_act=act)
+    _close(x, want, 1e-6)
+    assert torch.equal(act, x.to(dtype))
+    z = act.cpu().double() @ router[:n].double().T + bias.double()
+    for t in range(T):
+        wi, ww = R.route(z[t], top)
+        assert ids[t].tolist() == wi.tolist()
+        assert (wts[t].cpu().double() - ww).abs().max() < 1e-5
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("E,N,C,taps,top", [(64, 48, 40, 4, 0), (51, 9, 9, 2, 3), (640, 100, 33, 1, 2), (2052, 31, 0, 3, 4), (8, 1, 1, 7, 1)])
+def test_products_that_form_the_normed_sum_and_convolve_their_rows(dtype, E, N, C, taps, top):
+    """Several tokens one after another: the summed row is handed on, every row of the product sees it, and the first C
+    rows pass a convolution whose tail moves on from call to call; a second product shares the row."""
+    from cold_compress_b200 import _lib
+    ops = _ops()
+    g = torch.Generator().manual_seed(E)
+    T = 9
+    xs, ys = torch.randn(T, E, generator=g), torch.randn(T, max(top, 1), E, generator=g)
+    wts = torch.softmax(torch.randn(T, max(top, 1), generator=g), -1)
+    gain = torch.randn(E, generator=g) * 0.5
+    W, W2 = (torch.randn(N, E, generator=g) * E ** -0.5).to(dtype), (torch.randn(5, E, generator=g) * E ** -0.5).to(dtype)
+    table = torch.randn(C, taps, generator=g)
+    mixed = (ys.double() * wts.double()[:, :, None]).sum(1) if top else ys[:, 0].double()
+    stream = xs.double() + R.rms_around_one(mixed, gain.double(), 1e-4)
+    rounded = stream.to(torch.float32).to(dtype).double()
+    want = rounded @ W.double().T
+    want2 = rounded @ W2.double().T
+    if C:
+        want = torch.cat([R.silu(R.causal_conv(want[:, :C], table.double())), want[:, C:]], 1)
+    tail = torch.zeros(taps - 1, C, device=DEV)
+    for t in range(T):
+        out, out2, total = torch.empty(1, N, device=DEV), torch.empty(1, 5, device=DEV), torch.empty(1, E, device=DEV)
+        pre = ops.output_norm_row(xs[t:t + 1].to(DEV), ys[t].to(DEV), gain.to(DEV), 1e-4, 1.0, total, wts=wts[t].to(DEV) if top else None)
+        ops.gemv_multi([(None, W.to(DEV), out), (None, W2.to(DEV), out2)], pre=pre,
+                       conv=(table.to(DEV), tail, _lib.ACT_SILU) if C else None)
+        _close(total[0], stream[t], 1e-6)
+        rel = 2e-5 if dtype == torch.float32 else 2e-2
+        assert (out[0].cpu().double() - want[t]).abs().max() < rel * want.abs().max()
+        assert (out2[0].cpu().double() - want2[t]).abs().max() < rel * want2.abs().max()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,V,N", [(4, 12, 48), (1, 1, 3), (9, 70, 20), (8, 128, 33)])
+def test_product_of_normed_and_gated_heads(dtype, H, V, N):
+    from cold_compress_b200 import _lib
+    ops = _ops()
+    g = torch.Generator().manual_seed(H * V)
+    y, gate, w = torch.randn(1, H * V, generator=g) * 0.01, torch.randn(1, H * V + 4, generator=g) * 2, torch.randn(V, generator=g)
+    W, out = (torch.randn(N, H * V, generator=g) * (H * V) ** -0.5).to(dtype), torch.empty(1, N, device=DEV)
+    heads = R.rms_plain(y.double().view(H, V), w.double(), 1e-4) * R.silu(gate[:, 3:3 + H * V].double().view(H, V))
+    ops.gemv_multi([(None, W.to(DEV), out)], pre=ops.gated_heads_row(y.to(DEV), w.to(DEV), gate.to(DEV)[:, 3:3 + H * V], _lib.ACT_SILU, 1e-4))
+    _close(out[0], W.double() @ heads.reshape(-1), 1e-5 if dtype == torch.float32 else 2e-2)
+
+
+def test_a_large_router_takes_a_launch_of_its_own():
+    from cold_compress_b200.nobodra import NobodraBlock
+    cfg = make_config(default_layers())
+    W = random_weights(cfg, seed=15)
+    tokens = torch.randint(0, cfg["vocab"], (30,), generator=torch.Generator().manual_seed(16)).tolist()
+    want = reference_logits(cfg, W, tokens)
+    model = build_model(cfg, W, torch.float32, 30)
+    launches = model.kernels_per_token()
+    keep, NobodraBlock.ROUTER_BYTES = NobodraBlock.ROUTER_BYTES, 0
+    try:
+        assert model.kernels_per_token() == launches + 2 * 3
+        got = run_portions(model, tokens, (10,) + (1,) * 20)
+    finally:
+        NobodraBlock.ROUTER_BYTES = keep
+    assert row_error(got, want).max() < fp32_tolerance(cfg, W, tokens, want)
+
+
+def test_bad_arguments_are_errors_not_launches():
+    from cold_compress_b200 import _lib
+    ops = _ops()
+    x = torch.zeros(1, 8, device=DEV)
+    W, w = torch.zeros(4, 8, device=DEV), torch.zeros(8, device=DEV)
+    with pytest.raises(AssertionError):
+        ops.output_norm_row(x, x.clone(), w, 1e-5, 1.0, x)                      # other CTAs would read what one has written
+    pre = ops.output_norm_row(x, x.clone(), w, 1e-5, 1.0, torch.zeros(1, 8, device=DEV))
+    with pytest.raises(_lib.CcError, match="shared input row"):                 # the row is handed on by the first job's CTA
+        ops.gemv_multi([(x, W, torch.zeros(1, 4, device=DEV)), (None, W, torch.zeros(1, 4, device=DEV))], pre=pre)
+    with pytest.raises(_lib.CcError, match="post_norm_route"):
+        ops.post_norm_route(x, x.clone(), w, 1e-5, 1.0, W, torch.zeros(2, device=DEV), torch.zeros(1, 3, dtype=torch.int32, device=DEV),
+                            torch.zeros(1, 3, device=DEV))
+
+
 # ----------------------------------------------------------------------------------------------- router and experts
 
 @pytest.mark.parametrize("n,top", [(1, 1), (6, 2), (12, 12), (40, 5), (70, 1)])
