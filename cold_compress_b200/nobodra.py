@@ -174,12 +174,12 @@ class NobodraBlock(nn.Module):
         E, m, mlp = cfg.dim, layer["mixer"], layer.get("mlp")
         self.kind = layer["type"]
         if self.kind == "delta":
-            self.mixer = DeltaMixer(E, int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]), cfg.norm_eps, dtype)
+            self.mixer = DeltaMixer(E, int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m["vdim"]), int(m.get("conv", 1)), cfg.norm_eps, dtype)
         else:
             rot = m.get("rot") or {}
             if int(m.get("vdim", m["dim"])) != int(m["dim"]):
                 raise ValueError("values that are the projected keys are as wide as the keys")
-            self.mixer = KeyValueAttention(E, int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), float(m["scale"]),
+            self.mixer = KeyValueAttention(E, int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), float(m["scale"]),
                                            int((m.get("mask") or {}).get("size", 0)), float(rot.get("base", 10000.0)),
                                            int(rot.get("dims", 0)), cfg.norm_eps, dtype)
         self.norm1 = OutputNorm(E, cfg.norm_eps)
@@ -407,7 +407,9 @@ class NobodraTransformer(nn.Module):
                 nk, nv, taps = r.kv_heads * r.head_dim, r.heads * r.v_dim, r.conv.taps
                 put(m.w_in, _padded_rows([get(q + "q", (nk, E)), get(q + "k", (nk, E)), get(q + "v", (nv, E)), get(q + "b", (r.heads, E)),
                                           get(q + "a", (r.heads, E)), get(q + "g", (nv, E))], m.w_in.shape[0]))
-                put(r.conv.weight, torch.cat([get(q + n + ".conv", (w, taps)).float() for n, w in (("q", nk), ("k", nk), ("v", nv))]))
+                # a checkpoint may leave out the table of a one-tap convolution: that is the identity
+                put(r.conv.weight, torch.cat([get(q + n + ".conv", (w, taps)).float() if taps > 1 or q + n + ".conv" in tensors else torch.ones(w, 1)
+                                              for n, w in (("q", nk), ("k", nk), ("v", nv))]))
                 put(r.A_log, get(q + "A_log", (r.heads,)).float())
                 put(r.dt_bias, get(q + "dt_bias", (r.heads,)).float())
                 put(r.norm_w, get(q + "norm", (r.v_dim,)).float())

@@ -484,7 +484,7 @@ def output_norm_row(x, y, w, eps, gain_offset, x_out, wts=None):
     p = _lib.CcSeqGemvPre()
     p.kind, p.x, p.y, p.w, p.x_out, p.eps, p.gain_offset = _lib.GEMV_PRE_OUTPUT_NORM, _p(x), _p(y), _p(w), _p(x_out), float(eps), float(gain_offset)
     p.wts, p.top = _p(wts), 0 if wts is None else wts.numel()
-    p.length = E
+    p.length, p.tensors = E, (x, y, w, x_out, wts)      # alive until the launch
     return p
 
 
@@ -496,7 +496,7 @@ def gated_heads_row(y, w, gate, act, eps):
     gp, _ = _cols(_f32("gate", gate))
     assert gate.numel() == K and K % w.numel() == 0
     p.kind, p.y, p.w, p.gate, p.gate_act, p.w_len, p.eps = _lib.GEMV_PRE_GATED_HEADS, _p(y), _p(w), gp, int(act), w.numel(), float(eps)
-    p.length = K
+    p.length, p.tensors = K, (y, w, gate)               # alive until the launch
     return p
 
 
