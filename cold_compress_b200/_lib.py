@@ -134,7 +134,7 @@ def check(rc: int, what: str = "") -> int:
 
 # --------------------------------------------------------------------------- libcc_b200_seq.so (include/cc_b200_seq.h)
 SEQ_SO_PATH = Path(os.environ.get("CC_B200_SEQ_LIB", PKG / "libcc_b200_seq.so"))
-SEQ_ABI_VERSION = 5
+SEQ_ABI_VERSION = 6
 DT_F32, DT_BF16 = 0, 1
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
 
@@ -198,11 +198,20 @@ GEMV_PRE_NONE, GEMV_PRE_OUTPUT_NORM, GEMV_PRE_GATED_HEADS = range(3)
 
 class CcSeqGemvPre(C.Structure):
     _fields_ = [(n, _i32) for n in ("kind", "top", "w_len", "gate_act")] + [(n, _vp) for n in ("x", "y", "wts", "w", "gate", "x_out")] + [
-        ("eps", _f32), ("gain_offset", _f32)]
+        ("eps", _f32), ("gain_offset", _f32), ("part_len", _i32)]
+
+
+class CcSeqBounded(C.Structure):
+    _fields_ = [("alpha", _vp), ("w", _vp), ("b", _vp)]
+
+
+class CcSeqBoundedSum(C.Structure):
+    _fields_ = [("x", _vp), ("y", _vp), ("ldy", _i64), ("out_norm", CcSeqBounded), ("mult", _f32), ("add", _vp), ("x_out", _vp),
+                ("next_norm", CcSeqBounded), ("h", _vp), ("act_dtype", _i32), ("rows", _vp), ("T", _i32), ("E", _i32)]
 
 
 class CcSeqGemvMulti(C.Structure):
-    _fields_ = [("job", CcSeqGemvJob * GEMV_MAX_JOBS), ("n_jobs", _i32), ("w_dtype", _i32), ("pre", CcSeqGemvPre)]
+    _fields_ = [("job", CcSeqGemvJob * GEMV_MAX_JOBS), ("n_jobs", _i32), ("w_dtype", _i32), ("pre", CcSeqGemvPre), ("post", CcSeqBoundedSum)]
 
 
 class CcSeqLatentPrep(C.Structure):
@@ -221,7 +230,7 @@ class CcSeqLatentDecode(C.Structure):
     _fields_ = [(n, _vp) for n in ("q", "k_new", "k_cache", "pos", "mask", "cache_cts", "input_pos", "y")] + [
         (n, _i32) for n in ("H", "Dk", "C", "L", "cache_dtype", "y_dtype")] + [("scale", _f32), ("append", _i32),
                                                                                ("workspace", _vp), ("workspace_bytes", C.c_uint64),
-                                                                               ("sink", _vp)]
+                                                                               ("sink", _vp), ("window", _i32)]
 
 
 class CcSeqWkv(C.Structure):
@@ -278,7 +287,8 @@ class CcSeqDeltaScan(C.Structure):
 class CcSeqQkvRope(C.Structure):
     _fields_ = [("inp", _vp), ("ld", _i64)] + [(n, _i32) for n in ("off_q", "off_k", "off_v", "H", "G", "Dk", "Dv")] + [
         ("q_norm_w", _vp), ("k_norm_w", _vp), ("eps", _f32), ("rot_dims", _i32), ("interleaved", _i32), ("inv_freq", _vp),
-        ("v_inv_freq", _vp), ("input_pos", _vp), ("q_out", _vp), ("k_out", _vp), ("v_out", _vp), ("out_dtype", _i32), ("T", _i32)]
+        ("v_inv_freq", _vp), ("input_pos", _vp), ("q_out", _vp), ("k_out", _vp), ("v_out", _vp), ("out_dtype", _i32), ("T", _i32),
+        ("q_bias", _vp), ("k_bias", _vp), ("v_bias", _vp), ("turn_gain", _f32)]
 
 
 SEQ_EXPORTS.update({
@@ -324,6 +334,23 @@ class CcSeqPostNorm(C.Structure):
 SEQ_EXPORTS.update({
     "cc_seq_post_norm": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp]),
     "cc_seq_post_norm_route": (C.c_int, [C.POINTER(CcSeqPostNorm), _vp, _vp, _i32, _i32, _vp, _vp, _vp]),
+})
+
+# ---- sixth part of the header: element-wise bounded norms, matrix memory with exponential gates (csrc/seq/cell_kernels.cu)
+MLSTM_AUTO, MLSTM_SCAN, MLSTM_CHUNKS = range(3)
+
+
+class CcSeqMlstm(C.Structure):
+    _fields_ = [(n, _vp) for n in ("q", "k", "v", "i_raw", "f_raw")] + [("ld", _i64), ("i_bias", _vp), ("f_bias", _vp)] + [
+        (n, _f32) for n in ("gate_cap", "q_scale", "den_eps")] + [(n, _vp) for n in ("state", "aux", "o")] + [
+        (n, _i32) for n in ("T", "H", "D", "V", "path")] + [("workspace", _vp), ("workspace_bytes", C.c_uint64)]
+
+
+SEQ_EXPORTS.update({
+    "cc_seq_bounded_sum": (C.c_int, [C.POINTER(CcSeqBoundedSum), _vp]),
+    "cc_seq_embed_bounded": (C.c_int, [_vp, _vp, _i32, C.POINTER(CcSeqBounded), _vp, C.POINTER(CcSeqBounded), _vp, _i32, _i32, _i32, _vp]),
+    "cc_seq_mlstm_workspace": (C.c_uint64, [_i32] * 5),
+    "cc_seq_mlstm": (C.c_int, [C.POINTER(CcSeqMlstm), _vp]),
 })
 
 _seq_lib = None

@@ -805,7 +805,8 @@ class KVCacheLatent(KVCacheFull):
     """The cache of a latent (low-rank) attention layer: one row per position, shared by all query heads, holding the
     normalised key/value latent followed by the rotated key part (`k_cache` [1, 1, L, rank + rot]).  There are no
     value rows: a row's first `rank` columns are its value in the absorbed one-token step, and prompt portions
-    up-project the rows they need.  Nothing is ever evicted (slot = position)."""
+    up-project the rows they need.  Nothing is evicted while the sequence fits (slot = position); with fewer slots than
+    positions the rows are a ring of the newest ones (slot = position mod L), for layers that look back at most L."""
 
     def __init__(self, max_batch_size, n_heads, head_dim, dtype=torch.bfloat16, **kwargs):
         if n_heads != 1:
@@ -814,7 +815,7 @@ class KVCacheLatent(KVCacheFull):
         self.register_buffer("v_cache", torch.zeros((max_batch_size, 1, 0, 0), dtype=dtype))
 
     def latent_rows(self, n):
-        """[n, rank + rot] view of the rows of positions 0 .. n-1."""
+        """[n, rank + rot] view of the first n slots: the rows of positions 0 .. n-1 until the ring wraps."""
         return self.k_cache[0, 0, :n]
 
     def sequence_step(self, *args, **kwargs):
@@ -825,11 +826,13 @@ class KVCacheLatent(KVCacheFull):
         from . import seq_ops
         seq_ops.cache_append(k_new, None, self.k_cache, None, self.pos, self.mask, self.cache_cts, input_pos)
 
-    def latent_step(self, q, k_new, input_pos, y, scale, sink=None):
+    def latent_step(self, q, k_new, input_pos, y, scale, sink=None, window=0):
         """One token: q fp32 [1, H, rank + rot] over the cached rows and k_new [1, 1, rank + rot], which is then stored;
-        y [1, H, rank].  `sink` (fp32 [H]): a logit per head whose exponential joins the softmax denominator.  Two
-        launches, positions read on the device (capturable in a graph)."""
+        y [1, H, rank].  `sink` (fp32 [H]): a logit per head whose exponential joins the softmax denominator.  `window` > 0:
+        only the newest `window` positions are keys.  Two launches, positions read on the device (capturable in a graph)."""
         from . import seq_ops
+        if window and window > self.max_cache_length:
+            raise _lib.CcError(f"cache keeps {self.max_cache_length} positions but the layer looks back {window}")
         H, C = q.shape[-2], y.shape[-1]
         key = ("latent", H, C, self.k_cache.device)
         ws = self._out.get("latent_ws")
@@ -837,13 +840,14 @@ class KVCacheLatent(KVCacheFull):
             nbytes = seq_ops.latent_decode_workspace_bytes(H, C, self.max_cache_length)
             ws = (key, torch.empty((nbytes + 3) // 4, dtype=torch.float32, device=self.k_cache.device))
             self._out["latent_ws"] = ws
-        seq_ops.latent_decode(q, k_new, self.k_cache, self.pos, self.mask, self.cache_cts, input_pos, y, scale, ws[1], sink=sink)
+        seq_ops.latent_decode(q, k_new, self.k_cache, self.pos, self.mask, self.cache_cts, input_pos, y, scale, ws[1], sink=sink, window=window)
         return y
 
 
 class RecurrentState(nn.Module):
     """What a sequence carries from token to token besides key/value rows: `vectors` fp32 [n_vectors, width]
-    (previous-token activations for a token shift, or the last inputs of a short convolution) and, for a layer with a
+    (previous-token activations for a token shift, the last inputs of a short convolution, or per head the key sum and
+    the running maximum of an exponentially gated memory) and, for a layer with a
     matrix-state recurrence, `matrix` fp32 [n_heads, head_dim, state_cols] (state_cols defaults to head_dim).  Fixed
     size whatever the sequence length; `reset` gives it back (all zero = the state before the first token).  Built
     through `get_cache_constructor("state")` like the caches."""

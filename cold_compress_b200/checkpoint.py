@@ -71,6 +71,9 @@ def _builtin():
     if "Nobodra" not in MODEL_REGISTRY:
         from .nobodra import NobodraTransformer
         register_model("Nobodra", NobodraTransformer.from_config)
+    if "Relanex" not in MODEL_REGISTRY:
+        from .relanex import RelanexTransformer
+        register_model("Relanex", RelanexTransformer.from_config)
 
 
 def is_checkpoint_folder(path) -> bool:

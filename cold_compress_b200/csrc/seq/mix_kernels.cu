@@ -661,6 +661,8 @@ __host__ __device__ inline int ld_stride(int width) {   // floats; a multiple of
 }
 __host__ __device__ inline int ld_keys_per_run(int L) { return LD_TK * ((L + LD_TK * 128 - 1) / (LD_TK * 128)); }   // at most 128 runs
 
+__device__ __forceinline__ int ld_first_key(const CcSeqLatentDecode& a, int p) { return a.window > 0 ? max(0, p - a.window + 1) : 0; }
+
 template <typename CT, int NC>
 __global__ void __launch_bounds__(LD_THREADS) latent_decode_kernel(const CcSeqLatentDecode a) {
     extern __shared__ float4 sml4[];
@@ -671,7 +673,7 @@ __global__ void __launch_bounds__(LD_THREADS) latent_decode_kernel(const CcSeqLa
     float* Ps = Ks + LD_TK * Dkp;           // [LD_HG][LD_TK]
     int* src = (int*)(Ps + LD_HG * LD_TK);  // [LD_TK] slot, -1 = not a key, -2 = the new row
     const int p = a.input_pos[0], kpr = ld_keys_per_run(a.L);
-    const int j_begin = blockIdx.x * kpr;
+    const int j_begin = ld_first_key(a, p) + blockIdx.x * kpr;
     if (j_begin > p) return;
     const int j_end = min(p, j_begin + kpr - 1);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -779,7 +781,7 @@ __global__ void __launch_bounds__(LC_WARPS * 32) latent_combine_kernel(const CcS
     __shared__ float red[LC_WARPS];
     const int h = blockIdx.x, C = a.C, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int p = a.input_pos[0], kpr = ld_keys_per_run(a.L);
-    const int runs = min(p / kpr + 1, (a.L + kpr - 1) / kpr);   // never more runs than the tile kernel has
+    const int runs = min((p - ld_first_key(a, p)) / kpr + 1, (a.L + kpr - 1) / kpr);   // never more runs than the tile kernel has
     const float* ws = (const float*)a.workspace;
     const size_t stride = (size_t)a.H * (2 + C);
     const float* mine = ws + (size_t)h * (2 + C);
@@ -910,15 +912,28 @@ __device__ __forceinline__ void gemv_output_norm_row(const CcSeqGemvPre& p, floa
 
 template <typename WT>
 __device__ __forceinline__ void gemv_gated_heads_row(const CcSeqGemvPre& p, float* xs, int K, const WT* W) {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, V = p.w_len;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, V = p.part_len > 0 ? p.part_len : p.w_len;
     for (int h = warp; h < K / V; h += 8) {
         const float* y = p.y + (size_t)h * V;
         const float* gate = p.gate + (size_t)h * V;
+        const float* w = p.w + (h * V) % p.w_len;
         float ss = 0.f;
         for (int e = lane; e < V; e += 32) ss = fmaf(y[e], y[e], ss);
         const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)V + p.eps);
-        for (int e = lane; e < V; e += 32) xs[h * V + e] = round_to(y[e] * rinv * p.w[e] * unit_act(gate[e], p.gate_act), W);
+        for (int e = lane; e < V; e += 32) xs[h * V + e] = round_to(y[e] * rinv * w[e] * unit_act(gate[e], p.gate_act), W);
     }
+}
+
+// The way out of a product whose row n is a sublayer's result for channel n: bounded norm, sum into the stream, the next
+// sublayer's bounded norm (the arithmetic of bounded_sum_kernel).  The channel belongs to this row alone.
+__device__ __forceinline__ void bounded_row(const CcSeqBoundedSum& p, int n, float y) {
+    float s = fmaf(p.mult, fmaf(p.out_norm.w[n], tanhf(*p.out_norm.alpha * y), p.out_norm.b[n]), p.x[n]);
+    if (p.add != nullptr) s += p.add[n];
+    if (p.x_out != nullptr) p.x_out[n] = s;
+    if (p.h == nullptr) return;
+    const float v = fmaf(p.next_norm.w[n], tanhf(*p.next_norm.alpha * s), p.next_norm.b[n]);
+    if (p.act_dtype == CC_DT_BF16) stf((bf16*)p.h, n, v);
+    else stf((float*)p.h, n, v);
 }
 
 template <typename WT, int PRE>
@@ -1007,7 +1022,8 @@ __global__ void __launch_bounds__(256) gemv_multi_kernel(const CcSeqGemvMulti g)
         if (taps > 1) jb.tail[(size_t)(taps - 2) * C + n] = acc;
         acc = unit_act(fmaf(cw[taps - 1], acc, c), jb.conv_act);
     }
-    ((float*)jb.out)[n] = acc;
+    if (j == 0 && g.post.x != nullptr) bounded_row(g.post, n, acc);
+    if (jb.out != nullptr) ((float*)jb.out)[n] = acc;
 }
 
 template <int TB, int CH>
@@ -1251,7 +1267,7 @@ uint64_t cc_seq_latent_decode_workspace(int32_t H, int32_t C, int32_t L) {
 
 int cc_seq_latent_decode(const CcSeqLatentDecode* a, void* stream) {
     if (!a || !a->q || !a->k_new || !a->k_cache || !a->pos || !a->input_pos || !a->y || a->H < 1 || a->Dk < 1 || a->C < 1 ||
-        a->C > a->Dk || a->L < 1)
+        a->C > a->Dk || a->L < 1 || a->window < 0 || (a->window > 0 && a->L < a->window))
         return fail(CC_SEQ_ERR_INVALID_ARG, "latent_decode: bad argument");
     if (!a->workspace || a->workspace_bytes < cc_seq_latent_decode_workspace(a->H, a->C, a->L))
         return fail(CC_SEQ_ERR_INVALID_ARG, "latent_decode: workspace missing or too small");
@@ -1272,7 +1288,7 @@ int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream) {
     int blocks = 0, kmax = 0;
     for (int j = 0; j < g->n_jobs; ++j) {
         const CcSeqGemvJob& b = g->job[j];
-        if (!b.W || !b.out || b.N < 1 || b.K < 1 || b.kind < CC_ACT_NONE || b.kind > CC_ACT_LAST ||
+        if (!b.W || (!b.out && !(j == 0 && g->post.x)) || b.N < 1 || b.K < 1 || b.kind < CC_ACT_NONE || b.kind > CC_ACT_LAST ||
             ((b.kind != CC_ACT_NONE || b.off_up >= 0) && b.x_dtype != CC_DT_F32))
             return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad job");
         if (b.conv_rows < 0 || b.conv_rows > b.N || (b.conv_rows > 0 && (!b.conv_w || b.taps < 1 || (b.taps > 1 && !b.tail) ||
@@ -1281,6 +1297,7 @@ int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream) {
         if (!b.x) {
             const bool ok = p.kind == CC_GEMV_PRE_OUTPUT_NORM ? p.x && p.y && p.w && p.x_out && p.x_out != p.x && p.top >= 0 && (p.top == 0 || p.wts) :
                             p.kind == CC_GEMV_PRE_GATED_HEADS ? p.y && p.w && p.gate && p.w_len >= 1 && b.K % p.w_len == 0 &&
+                                                                p.part_len >= 0 && (p.part_len == 0 || p.w_len % p.part_len == 0) &&
                                                                 p.gate_act >= CC_ACT_NONE && p.gate_act <= CC_ACT_LAST : false;
             // CTA 0 belongs to job 0: it is the one that hands the summed row on
             if (!ok || b.kind != CC_ACT_NONE || b.off_up >= 0 || g->job[0].x || b.K != g->job[0].K)
@@ -1289,6 +1306,10 @@ int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream) {
         blocks += (b.N + 7) / 8;
         kmax = b.K > kmax ? b.K : kmax;
     }
+    const CcSeqBoundedSum& q = g->post;
+    if (q.x && (!q.out_norm.w || !q.out_norm.b || !q.out_norm.alpha || (!q.x_out && !q.h) ||
+                (q.h && (!q.next_norm.w || !q.next_norm.b || !q.next_norm.alpha || (q.act_dtype != CC_DT_F32 && q.act_dtype != CC_DT_BF16)))))
+        return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: bad way out");
     if (p.kind < CC_GEMV_PRE_NONE || p.kind > CC_GEMV_PRE_GATED_HEADS) return fail(CC_SEQ_ERR_INVALID_ARG, "gemv_multi: unknown shared input row");
     const size_t smem = sizeof(float) * (size_t)((kmax + 3) & ~3);
     if (smem > 200 * 1024) return fail(CC_SEQ_ERR_UNSUPPORTED_SHAPE, "gemv_multi: input longer than 51200");

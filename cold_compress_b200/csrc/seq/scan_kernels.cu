@@ -532,21 +532,27 @@ __global__ void qkv_rope_kernel(const CcSeqQkvRope a) {
         const int Dk = a.Dk, head = isq ? hh : hh - a.H;
         const float* row = in + (isq ? a.off_q : a.off_k) + (size_t)head * Dk;
         const float* nw = isq ? a.q_norm_w : a.k_norm_w;
+        const float* bias = isq ? a.q_bias : a.k_bias;
+        if (bias != nullptr) bias += (size_t)head * Dk;
+        const float gain = a.turn_gain != 0.f ? a.turn_gain : 1.f;
+        auto raw = [&](int d) { return bias != nullptr ? row[d] + bias[d] : row[d]; };
         float rinv = 1.f;
         if (nw != nullptr) {
             float ss = 0.f;
-            for (int d = lane; d < Dk; d += 32) ss = fmaf(row[d], row[d], ss);
+            for (int d = lane; d < Dk; d += 32) { const float v = raw(d); ss = fmaf(v, v, ss); }
             rinv = 1.0f / sqrtf(warp_sum(ss) / (float)Dk + a.eps);
         }
         float* qo = isq ? a.q_out + (t * a.H + head) * Dk : nullptr;
         OT* ko = isq ? nullptr : (OT*)a.k_out + (t * a.G + head) * Dk;
-        auto val = [&](int d) { return nw != nullptr ? row[d] * rinv * nw[d] : row[d]; };
+        auto val = [&](int d) { return nw != nullptr ? raw(d) * rinv * nw[d] : raw(d); };
         auto put = [&](int d, float v) { if (isq) qo[d] = v; else stf(ko, d, v); };
         for (int i = lane; i < a.rot_dims / 2; i += 32) {
             int d0, d1;
             pair_index(i, a.rot_dims, a.interleaved, d0, d1);
             float s, c;
             sincosf(pos * a.inv_freq[i], &s, &c);
+            s *= gain;
+            c *= gain;
             const float u = val(d0), v = val(d1);
             put(d0, u * c - v * s);
             put(d1, v * c + u * s);
@@ -555,6 +561,8 @@ __global__ void qkv_rope_kernel(const CcSeqQkvRope a) {
     } else {
         const int head = hh - a.H - a.G, Dv = a.Dv;
         const float* row = in + a.off_v + (size_t)head * Dv;
+        const float* bias = a.v_bias != nullptr ? a.v_bias + (size_t)head * Dv : nullptr;
+        auto raw = [&](int d) { return bias != nullptr ? row[d] + bias[d] : row[d]; };
         OT* vo = (OT*)a.v_out + (t * a.G + head) * Dv;
         if (a.v_inv_freq != nullptr) {
             for (int i = lane; i < Dv / 2; i += 32) {
@@ -562,13 +570,13 @@ __global__ void qkv_rope_kernel(const CcSeqQkvRope a) {
                 pair_index(i, Dv, a.interleaved, d0, d1);
                 float s, c;
                 sincosf(pos * a.v_inv_freq[i], &s, &c);
-                const float u = row[d0], v = row[d1];
+                const float u = raw(d0), v = raw(d1);
                 stf(vo, d0, u * c - v * s);
                 stf(vo, d1, v * c + u * s);
             }
-            if ((Dv & 1) && lane == 0) stf(vo, Dv - 1, row[Dv - 1]);
+            if ((Dv & 1) && lane == 0) stf(vo, Dv - 1, raw(Dv - 1));
         } else {
-            for (int d = lane; d < Dv; d += 32) stf(vo, d, row[d]);
+            for (int d = lane; d < Dv; d += 32) stf(vo, d, raw(d));
         }
     }
 }

@@ -880,7 +880,8 @@ static int check_attn(const CcSeqAttn* a) {
     if (a->Dk > 256 || a->Dv > 256) return fail(CC_SEQ_ERR_UNSUPPORTED_SHAPE, "attention: head sizes above 256");
     if (a->keep_first < 0 || (a->keep_first > 0 && a->L <= a->keep_first) || a->softcap < 0.f || (a->dist_a && !a->dist_b))
         return fail(CC_SEQ_ERR_INVALID_ARG, "attention: bad kept-first count, soft cap or distance penalty");
-    if (a->window > 0 && a->L < a->window + a->keep_first)
+    // rows that are read only (no fill mask: not a cache) may be fewer than the window: a missing position is not a key
+    if (a->window > 0 && a->mask && a->L < a->window + a->keep_first)
         return fail(CC_SEQ_ERR_INVALID_ARG, "attention: cache capacity below the window plus the kept first positions");
     if (a->block < 0 || (a->block > 0 && (a->window > 0 || a->L < a->block)))
         return fail(CC_SEQ_ERR_INVALID_ARG, "attention: a block mask needs a cache of at least one block and no window");

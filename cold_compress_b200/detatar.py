@@ -197,7 +197,8 @@ class LatentAttention(nn.Module):
     [dim unrotated | rot_dim rotated].  Keys: per head `[W_uk c | rot(k_r)]` with `c = rms_norm(first kv_rank rows of
     W_dkv h)` and `k_r` the last rot_dim rows, shared by all heads; values `W_uv c`.  Options: `gated` multiplies each
     head's output by sigmoid of one row of `W_g h`; `sink` adds exp of a learned logit per head to the softmax
-    denominator; `interleaved` pairs rotary dimensions (2i, 2i + 1) instead of (i, i + dims / 2).
+    denominator; `interleaved` pairs rotary dimensions (2i, 2i + 1) instead of (i, i + dims / 2); `rot_dim` 0 = no rotated
+    part; `window` > 0 limits query i to keys j with i - j < window (the cache may then be a ring of one window).
 
     Only `[c | rot(k_r)]` is cached.  A prompt portion up-projects the cached latents of the earlier positions
     (tensor-core product) and attends over per-head rows; a single token uses the absorbed form instead: the query
@@ -206,13 +207,13 @@ class LatentAttention(nn.Module):
 
     def __init__(self, dim: int, heads: int, head_dim: int, rot_dim: int, v_dim: int, q_rank: int, kv_rank: int,
                  scale: float, rot_base: float, rot_dims: int, eps: float, dtype, gated: bool = True, sink: bool = False,
-                 interleaved: bool = False):
+                 interleaved: bool = False, window: int = 0):
         super().__init__()
         if rot_dims > rot_dim or rot_dims % 2:
             raise ValueError("rotary dims must be even and at most the rotated width")
         self.dim, self.heads, self.head_dim, self.rot_dim, self.v_dim = dim, heads, head_dim, rot_dim, v_dim
         self.q_rank, self.kv_rank, self.scale, self.rot_dims, self.eps = q_rank, kv_rank, float(scale), rot_dims, eps
-        self.gated, self.interleaved = bool(gated), bool(interleaved)
+        self.gated, self.interleaved, self.window = bool(gated), bool(interleaved), int(window)
         # rows of the fused input projection: query part (down-projection, or all query heads when q_rank == 0) | dkv | g | padding
         self.q_rows = q_rank if q_rank else heads * (head_dim + rot_dim)
         self.w_in = _zeros(_pad16(self.q_rows + kv_rank + rot_dim + (heads if gated else 0)), dim, dtype=dtype)
@@ -256,26 +257,30 @@ class LatentAttention(nn.Module):
         else:
             q = a[:, :Q]      # the query heads are columns of the fused projection (fp32), rotated in place
         qf = torch.empty(1, H, C + R, dtype=torch.float32, device=dev)
-        seq_ops.rope_heads(q, ip, self.inv_freq, H, D + R, D, R, self.rot_dims, tail=qf, tail_off=C, interleaved=self.interleaved)
+        if R:
+            seq_ops.rope_heads(q, ip, self.inv_freq, H, D + R, D, R, self.rot_dims, tail=qf, tail_off=C, interleaved=self.interleaved)
         seq_ops.head_gemv(self.w_uk_t, q, D + R, qf, C + R)
         ctx = torch.empty(1, H, C, dtype=dt, device=dev)
-        cache.latent_step(qf, krow, ip, ctx, self.scale, sink=self.sink)
+        cache.latent_step(qf, krow, ip, ctx, self.scale, sink=self.sink, window=self.window)
         y = torch.empty(1, H * V, dtype=dt, device=dev)
         seq_ops.head_gemv(self.w_ukv[H * D:].view(H, V, C), ctx, C, y, V,
                           gate=a[0, Q + C + R:Q + C + R + H] if self.gated else None)
         return y
 
     def forward(self, hs_act: Tensor, ip: Tensor, cache, one_token_kernel: bool = True) -> Tensor:
-        T, dev, dt = hs_act.shape[0], hs_act.device, self.w_in.dtype
-        H, D, R, V, C = self.heads, self.head_dim, self.rot_dim, self.v_dim, self.kv_rank
-        if T == 1 and one_token_kernel and self.absorbed_fits():
+        if hs_act.shape[0] == 1 and one_token_kernel and self.absorbed_fits():
             jobs, outs = self.first_jobs(hs_act)
             seq_ops.gemv_multi(jobs)
             y, out = self.finish(outs, ip, cache), _out(self.w_o)
             seq_ops.gemv_multi([(y, self.w_o, out)])
             return out
+        return _proj(self.expanded(_proj(hs_act, self.w_in), ip, cache), self.w_o)
+
+    def expanded(self, a: Tensor, ip: Tensor, cache) -> Tensor:
+        """A prompt portion, from the fused projection's fp32 rows to the input of the output projection [T, heads * v_dim]."""
+        T, dev, dt = a.shape[0], a.device, self.w_in.dtype
+        H, D, R, V, C = self.heads, self.head_dim, self.rot_dim, self.v_dim, self.kv_rank
         Q = self.q_rows
-        a = _proj(hs_act, self.w_in)
         cq = torch.empty(T, self.q_rank, dtype=dt, device=dev) if self.q_rank else None
         krow = torch.empty(T, 1, C + R, dtype=dt, device=dev)
         lat_new = torch.empty(T, C, dtype=dt, device=dev)     # contiguous latents for the up-projection
@@ -284,25 +289,29 @@ class LatentAttention(nn.Module):
         q = _proj(cq, self.w_uq) if self.q_rank else a[:, :Q].contiguous()             # fp32 [T, H * (D + R)]
         gate = a[:, Q + C + R:Q + C + R + H]
         p0 = int(ip.item())      # a prompt portion sizes its expanded rows on the host (one read per layer step)
-        seq_ops.rope_heads(q, ip, self.inv_freq, H, D + R, D, R, self.rot_dims, interleaved=self.interleaved)
+        if R:
+            seq_ops.rope_heads(q, ip, self.inv_freq, H, D + R, D, R, self.rot_dims, interleaved=self.interleaved)
         kv_new = _mm(lat_new, self.w_ukv)
         k_new = torch.empty(T, H, D + R, dtype=dt, device=dev)
         v_new = torch.empty(T, H, V, dtype=dt, device=dev)
+        window = self.window if p0 + T > self.window else 0      # 0: nothing lies outside the window yet
         if p0 > 0:
-            lat_old = cache.latent_rows(p0)
+            # row j of the old rows must hold position j (mod their number): the filled slots, or a whole ring
+            n_old = cache.max_cache_length if window else p0
+            lat_old = cache.latent_rows(n_old)
             kv_old = _mm(lat_old[:, :C].contiguous(), self.w_ukv)
-            k_old = torch.empty(H, p0, D + R, dtype=dt, device=dev)
-            v_old = torch.empty(H, p0, V, dtype=dt, device=dev)
-            pos_old = cache.pos[0, 0, :p0]
+            k_old = torch.empty(H, n_old, D + R, dtype=dt, device=dev)
+            v_old = torch.empty(H, n_old, V, dtype=dt, device=dev)
+            pos_old = cache.pos[0, 0, :n_old]
         else:
             lat_old = kv_old = k_old = v_old = pos_old = None
         seq_ops.latent_expand(kv_old, kv_new, lat_old, krow.view(T, C + R), k_old, v_old, k_new, v_new, H, D, V, R, C)
         y = torch.empty(T, H, V, dtype=dt, device=dev)
-        seq_ops.attention_rows(q.view(T, H, D + R), k_new, v_new, k_old, v_old, pos_old, ip, y, self.scale, sink=self.sink)
+        seq_ops.attention_rows(q.view(T, H, D + R), k_new, v_new, k_old, v_old, pos_old, ip, y, self.scale, window=window, sink=self.sink)
         cache.sequence_append(krow, ip)
         if self.gated:
             seq_ops.head_gate(y, gate)
-        return _proj(y.view(T, H * V), self.w_o)
+        return y.view(T, H * V)
 
 
 class GatedMLP(nn.Module):

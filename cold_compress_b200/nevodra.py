@@ -42,6 +42,16 @@ FEED_FORWARDS = ("dense", "moe")
 
 # --------------------------------------------------------------------------------------------- configuration
 
+def loop_runs(n: int, start: int, stop: int, times: int):
+    """[(layer index, pass number or None)] of n layers in running order: layers start .. stop-1 `times` times in a row."""
+    if stop <= start:
+        return [(i, None) for i in range(n)]
+    out = [(i, None) for i in range(start)]
+    for t in range(times):
+        out += [(i, t) for i in range(start, stop)]
+    return out + [(i, None) for i in range(stop, n)]
+
+
 @dataclass
 class NevodraArgs:
     vocab_size: int
@@ -70,14 +80,7 @@ class NevodraArgs:
         self.n_layer = len(self.runs())
 
     def runs(self):
-        """[(layer index, pass number or None)] in running order: layers start .. stop-1 `times` times in a row."""
-        n = len(self.layers)
-        if self.loop_stop <= self.loop_start:
-            return [(i, None) for i in range(n)]
-        out = [(i, None) for i in range(self.loop_start)]
-        for t in range(self.loop_times):
-            out += [(i, t) for i in range(self.loop_start, self.loop_stop)]
-        return out + [(i, None) for i in range(self.loop_stop, n)]
+        return loop_runs(len(self.layers), self.loop_start, self.loop_stop, self.loop_times)
 
     @classmethod
     def from_config(cls, cfg: Dict[str, Any]):

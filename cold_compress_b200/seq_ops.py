@@ -427,14 +427,15 @@ def latent_decode_workspace_bytes(H, C, L) -> int:
     return int(_lib.load_seq().cc_seq_latent_decode_workspace(int(H), int(C), int(L)))
 
 
-def latent_decode(q, k_new, k_cache, pos, mask, cache_cts, input_pos, y, scale, workspace, append=True, sink=None):
+def latent_decode(q, k_new, k_cache, pos, mask, cache_cts, input_pos, y, scale, workspace, append=True, sink=None, window=0):
     """Absorbed one-token latent attention: q fp32 [1, H, Dk] over rows k_cache [.., L, Dk] and k_new [.., Dk] (the newest
-    key, appended when asked); y [1, H, C] = weighted sums of the rows' first C columns."""
+    key, appended when asked); y [1, H, C] = weighted sums of the rows' first C columns.  window > 0: only the newest `window`
+    positions are keys."""
     _need(("q", q, torch.float32), ("k_new", k_new, k_cache.dtype), ("k_cache", k_cache, None), ("pos", pos, torch.int32),
           ("mask", mask, torch.bool), ("cache_cts", cache_cts, torch.int32), ("input_pos", input_pos, torch.int32), ("y", y, None),
           ("workspace", workspace, None), ("sink", sink, torch.float32))
     a = _lib.CcSeqLatentDecode()
-    a.sink = _p(sink)
+    a.sink, a.window = _p(sink), int(window)
     a.q, a.k_new, a.k_cache, a.pos, a.mask, a.cache_cts = _p(q), _p(k_new), _p(k_cache), _p(pos), _p(mask), _p(cache_cts)
     a.input_pos, a.y = _p(input_pos), _p(y)
     a.H, a.Dk, a.C, a.L = q.shape[-2], q.shape[-1], y.shape[-1], k_cache.shape[-2]
@@ -444,11 +445,13 @@ def latent_decode(q, k_new, k_cache, pos, mask, cache_cts, input_pos, y, scale, 
     _lib.check_seq(_lib.load_seq().cc_seq_latent_decode(C.byref(a), _stream()), "cc_seq_latent_decode")
 
 
-def gemv_multi(jobs, pre=None, conv=None):
+def gemv_multi(jobs, pre=None, conv=None, post=None):
     """Up to six one-token products in one launch.  jobs: (x, w, out) or (src, w, out, kind, off_gate, off_up) where the
     input is built from the fp32 row `src` as act(src[off_gate + k]) * src[off_up + k]; out fp32 [1, N].  x = None: the
     launch's shared row `pre` (output_norm_row or gated_heads_row), which every CTA forms for itself.  conv = (table
-    [C, taps], tail [taps - 1, C], act): the first C rows of job 0 pass that short convolution, whose tail moves on."""
+    [C, taps], tail [taps - 1, C], act): the first C rows of job 0 pass that short convolution, whose tail moves on.
+    post = bounded_way_out(...): job 0's rows are a sublayer's result and join the stream on their way out (its out may be
+    None)."""
     g = _lib.CcSeqGemvMulti()
     g.n_jobs = len(jobs)
     assert 1 <= len(jobs) <= _lib.GEMV_MAX_JOBS
@@ -459,12 +462,15 @@ def gemv_multi(jobs, pre=None, conv=None):
         _need(("x", x, None), ("w", w, jobs[0][1].dtype), ("out", out, torch.float32))
         N, K = w.shape
         built = kind != _lib.ACT_NONE or off_up >= 0
-        assert out.numel() == N and (pre.length == K if x is None else x.numel() >= max(off_gate, off_up) + K if built else x.numel() == K)
+        assert (out is None if j == 0 and post is not None and out is None else out.numel() == N) and (pre.length == K if x is None else x.numel() >= max(off_gate, off_up) + K if built else x.numel() == K)
         b = g.job[j]
         b.x, b.W, b.out = _p(x), _p(w), _p(out)
         b.x_dtype, b.kind, b.off_gate, b.off_up, b.N, b.K = _dt(x) if x is not None else _lib.DT_F32, int(kind), int(off_gate), int(off_up), N, K
     if pre is not None:
         g.pre = pre
+    if post is not None:
+        assert post.E == jobs[0][1].shape[0]
+        g.post = post
     if conv is not None:
         table, tail, act = conv
         _need(("table", table, torch.float32), ("tail", tail, torch.float32))
@@ -488,14 +494,17 @@ def output_norm_row(x, y, w, eps, gain_offset, x_out, wts=None):
     return p
 
 
-def gated_heads_row(y, w, gate, act, eps):
-    """Shared input row for gemv_multi: every part of len(w) entries of y [1, K] RMS-normed times w, times act(gate [1, K])."""
+def gated_heads_row(y, w, gate, act, eps, part=None):
+    """Shared input row for gemv_multi: every part of `part` (default len(w)) entries of y [1, K] RMS-normed, times w (repeated
+    over the row), times act(gate [1, K])."""
     _need(("y", y, torch.float32), ("w", w, torch.float32))
     p = _lib.CcSeqGemvPre()
     K = y.numel()
     gp, _ = _cols(_f32("gate", gate))
     assert gate.numel() == K and K % w.numel() == 0
     p.kind, p.y, p.w, p.gate, p.gate_act, p.w_len, p.eps = _lib.GEMV_PRE_GATED_HEADS, _p(y), _p(w), gp, int(act), w.numel(), float(eps)
+    p.part_len = 0 if part is None else int(part)
+    assert part is None or w.numel() % part == 0
     p.length, p.tensors = K, (y, w, gate)               # alive until the launch
     return p
 
@@ -604,7 +613,10 @@ def gated_rms_groups(y, gate, gate_act, gate_first, w, out, groups, eps):
 
 
 def qkv_rope(src, off_q, off_k, off_v, H, G, Dk, Dv, q_norm_w, k_norm_w, eps, rot_dims, interleaved, inv_freq, v_inv_freq,
-             input_pos, q_out, k_out, v_out):
+             input_pos, q_out, k_out, v_out, bias=None, turn_gain=1.0):
+    """`bias`: fp32 [H * Dk + G * Dk + G * Dv] (q | k | v), added to the rows first; `turn_gain` multiplies the turned
+    entries of q and k."""
+    _need(("bias", bias, torch.float32))
     _need(("q_norm_w", q_norm_w, torch.float32), ("k_norm_w", k_norm_w, torch.float32), ("inv_freq", inv_freq, torch.float32),
           ("v_inv_freq", v_inv_freq, torch.float32), ("input_pos", input_pos, torch.int32), ("q_out", q_out, torch.float32),
           ("k_out", k_out, None), ("v_out", v_out, k_out.dtype))
@@ -615,6 +627,11 @@ def qkv_rope(src, off_q, off_k, off_v, H, G, Dk, Dv, q_norm_w, k_norm_w, eps, ro
     assert (rot_dims == 0 or inv_freq.numel() >= rot_dims // 2) and (v_inv_freq is None or (Dv % 2 == 0 and v_inv_freq.numel() >= Dv // 2))
     a.inv_freq, a.v_inv_freq, a.input_pos = _p(inv_freq), _p(v_inv_freq), _p(input_pos)
     a.q_out, a.k_out, a.v_out, a.out_dtype, a.T = _p(q_out), _p(k_out), _p(v_out), _dt(k_out), src.shape[0]
+    a.turn_gain = float(turn_gain)
+    if bias is not None:
+        nq, nk = a.H * a.Dk, a.G * a.Dk
+        assert bias.numel() == nq + nk + a.G * a.Dv
+        a.q_bias, a.k_bias, a.v_bias = bias.data_ptr(), bias.data_ptr() + 4 * nq, bias.data_ptr() + 4 * (nq + nk)
     _lib.check_seq(_lib.load_seq().cc_seq_qkv_rope(C.byref(a), _stream()), "cc_seq_qkv_rope")
 
 
@@ -721,3 +738,86 @@ def post_norm_route(x, y, w, eps, gain_offset, router, bias, ids, wts, x_act=Non
     a.act_dtype = _dt(router)
     _lib.check_seq(_lib.load_seq().cc_seq_post_norm_route(C.byref(a), _p(router), _p(bias), n, ids.shape[1], _p(ids), _p(wts), _stream()),
                    "cc_seq_post_norm_route")
+
+
+# ------------------------------------------------------------------------------------------------------------------
+# Sixth part of the C ABI (csrc/seq/cell_kernels.cu): element-wise bounded norms, a matrix memory with exponential gates.
+# A bounded norm is a triple (alpha fp32 [1], w fp32 [E], b fp32 [E]): w * tanh(alpha * v) + b.
+
+def _bounded(norm, E):
+    alpha, w, b = norm
+    _need(("alpha", alpha, torch.float32), ("w", w, torch.float32), ("b", b, torch.float32))
+    assert alpha.numel() == 1 and w.numel() == E and b.numel() == E
+    return _lib.CcSeqBounded(_p(alpha), _p(w), _p(b))
+
+
+def _bounded_args(x, mult, out_norm, add, x_out, next_norm, h):
+    _need(("x", x, torch.float32), ("add", add, torch.float32), ("x_out", x_out, torch.float32), ("h", h, None))
+    a = _lib.CcSeqBoundedSum()
+    E = x.shape[-1]
+    a.x, a.add, a.x_out, a.h, a.mult, a.E = _p(x), _p(add), _p(x_out), _p(h), float(mult), E
+    if out_norm is not None:
+        a.out_norm = _bounded(out_norm, E)
+    if h is not None:
+        a.next_norm, a.act_dtype = _bounded(next_norm, E), _dt(h)
+    return a
+
+
+def bounded_sum(x, y=None, out_norm=None, mult=1.0, add=None, x_out=None, next_norm=None, h=None, rows=None):
+    """s = x + mult * B_out(y) + add (y and add optional); x_out <- s (may be x); h <- B_next(s) in its dtype.  `rows` (int64)
+    selects rows of x, y and add; outputs are compact."""
+    _need(("rows", rows, torch.int64))
+    a = _bounded_args(x, mult, out_norm, add, x_out, next_norm, h)
+    a.y, a.ldy = _cols(_f32("y", y))
+    a.rows = _p(rows)
+    a.T = x.shape[0] if rows is None else rows.numel()
+    assert (y is None or y.shape == x.shape) and (add is None or add.shape == x.shape)
+    for out in (x_out, h):
+        assert out is None or out.shape == (a.T, a.E)
+    _lib.check_seq(_lib.load_seq().cc_seq_bounded_sum(C.byref(a), _stream()), "cc_seq_bounded_sum")
+
+
+def bounded_way_out(x, out_norm, mult, x_out=None, next_norm=None, h=None, add=None):
+    """The same for one token as the way out of a product (gemv_multi's `post`): its rows are y."""
+    assert x.numel() == x.shape[-1]
+    a = _bounded_args(x, mult, out_norm, add, x_out, next_norm, h)
+    a.T = 1
+    a.tensors = (x, out_norm, x_out, next_norm, h, add)     # alive until the launch
+    return a
+
+
+def embed_bounded(tokens, embed, emb_norm, x, next_norm=None, h=None):
+    """x = B_emb(embed[tokens]) fp32 [T, E]; h = B_next(x) in its dtype."""
+    _need(("tokens", tokens, torch.int32), ("embed", embed, None), ("x", x, torch.float32), ("h", h, None))
+    T, E = tokens.numel(), embed.shape[1]
+    assert x.shape == (T, E) and (h is None or h.shape == (T, E))
+    emb = _bounded(emb_norm, E)
+    nxt = _bounded(next_norm, E) if h is not None else None
+    _lib.check_seq(_lib.load_seq().cc_seq_embed_bounded(_p(tokens), _p(embed), _dt(embed), C.byref(emb), _p(x),
+                                                        C.byref(nxt) if nxt is not None else None, _p(h), _dt(h) if h is not None else _lib.DT_F32,
+                                                        T, E, _stream()), "cc_seq_embed_bounded")
+
+
+def mlstm(q, k, v, i_raw, f_raw, i_bias, f_bias, gate_cap, q_scale, state, aux, o, H, D, V, den_eps=1e-6, path=_lib.MLSTM_AUTO):
+    """Matrix memory over T tokens: q, k [T, H*D], v [T, H*V], i_raw, f_raw [T, H] column ranges of one fp32 row; state fp32
+    [H, D, V] and aux fp32 [H, D + 2] (key sum, running maximum, a counter that stays zero) carried; o fp32 [T, H*V]."""
+    _need(("i_bias", i_bias, torch.float32), ("f_bias", f_bias, torch.float32), ("state", state, torch.float32), ("aux", aux, torch.float32),
+          ("o", o, torch.float32))
+    a = _lib.CcSeqMlstm()
+    T = q.shape[0]
+    a.q, a.ld = _cols(_f32("q", q))
+    for name, t, cols in (("k", k, H * D), ("v", v, H * V), ("i_raw", i_raw, H), ("f_raw", f_raw, H)):
+        ptr, ld = _cols(_f32(name, t))
+        assert t.shape == (T, cols) and (ld == a.ld or T == 1), f"{name}: one row stride for all inputs"
+        setattr(a, name, ptr)
+    assert q.shape[1] == H * D and state.numel() == H * D * V and aux.numel() == H * (D + 2) and o.shape == (T, H * V)
+    assert i_bias.numel() == H and f_bias.numel() == H
+    a.i_bias, a.f_bias, a.gate_cap, a.q_scale, a.den_eps = _p(i_bias), _p(f_bias), float(gate_cap), float(q_scale), float(den_eps)
+    a.state, a.aux, a.o = _p(state), _p(aux), _p(o)
+    a.T, a.H, a.D, a.V, a.path = T, int(H), int(D), int(V), int(path)
+    lib = _lib.load_seq()
+    need = int(lib.cc_seq_mlstm_workspace(a.T, a.H, a.D, a.V, a.path))
+    ws = torch.empty((need + 15) // 16 * 4, dtype=torch.float32, device=o.device) if need else None
+    if need:
+        a.workspace, a.workspace_bytes = ws.data_ptr(), need
+    _lib.check_seq(lib.cc_seq_mlstm(C.byref(a), _stream()), "cc_seq_mlstm")

@@ -32,6 +32,7 @@ The mechanisms (`SumLayerNorm`, `ShortConv`, `StateSpaceMixer`, `BlockRotaryAtte
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
@@ -60,6 +61,26 @@ def _inv_freq(base: float, dims: int) -> Tensor:
     """base^(-2i / dims) for i < dims / 2, computed in float64 and rounded once."""
     i = torch.arange(0, max(dims // 2, 1), dtype=torch.float64)
     return torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / max(dims, 1)).to(torch.float32)
+
+
+def _stretched_inv_freq(base: float, dims: int, scaling: Optional[Dict[str, Any]]):
+    """(frequencies, gain on cos and sin) for a context stretched by scaling["factor"]: pairs that turn often within the
+    original context (index up to `lo`) keep their frequency, slow ones (from `hi`) are divided by the factor, those
+    between are blended linearly; the bounds are the pairs that make `fast` and `slow` turns over `original` positions.
+    float64, rounded once; (plain frequencies, 1) without scaling."""
+    if not scaling:
+        return _inv_freq(base, dims), 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def pair_of(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
+    i = torch.arange(0, max(dims // 2, 1), dtype=torch.float64)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / max(dims, 1))
+    return (f / factor * ramp + f * (1.0 - ramp)).to(torch.float32), 0.1 * math.log(factor) + 1.0
 
 
 # --------------------------------------------------------------------------------------------- configuration

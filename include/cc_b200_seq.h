@@ -21,7 +21,7 @@
 extern "C" {
 #endif
 
-#define CC_SEQ_ABI_VERSION 5
+#define CC_SEQ_ABI_VERSION 6
 
 #define CC_SEQ_OK                     0
 #define CC_SEQ_ERR_INVALID_ARG       -1
@@ -54,7 +54,7 @@ typedef struct CcSeqAttn {
     void* k_cache;             /* [G, L, Dk] cache dtype */
     void* v_cache;             /* [G, L, Dv] cache dtype */
     int32_t* pos;              /* [L] position held by each slot, -1 = empty */
-    uint8_t* mask;             /* [G, L] 1 = slot filled (may be NULL) */
+    uint8_t* mask;             /* [G, L] 1 = slot filled (may be NULL; then L may also be below the window) */
     int32_t* cache_cts;        /* [1] number of filled slots (may be NULL) */
     const int32_t* input_pos;  /* [1] */
     void* y;                   /* [T, H, Dv] y dtype */
@@ -243,6 +243,7 @@ int cc_seq_latent_expand(const CcSeqLatentExpand* a, void* stream);
  * newest key and, with `append`, is stored in slot position mod L (pos / mask / cache_cts as in CcSeqAttn).
  * y [H, C] = softmax(scale * q . row) weighted sum of the rows' first C columns.  Keys are addressed by position.
  * With `sink` (fp32 [H]) the softmax denominator also holds exp(sink[h]): a term without key or value.
+ * window > 0: only the newest `window` positions are keys (L >= window: the rows may be a ring of that size).
  */
 typedef struct CcSeqLatentDecode {
     const float* q;  const void* k_new;  void* k_cache;
@@ -253,6 +254,7 @@ typedef struct CcSeqLatentDecode {
     int32_t append;
     void* workspace;  uint64_t workspace_bytes;   /* cc_seq_latent_decode_workspace() bytes; needs no clearing */
     const float* sink;
+    int32_t window;
 } CcSeqLatentDecode;
 uint64_t cc_seq_latent_decode_workspace(int32_t H, int32_t C, int32_t L);
 int cc_seq_latent_decode(const CcSeqLatentDecode* a, void* stream);
@@ -265,9 +267,12 @@ int cc_seq_latent_decode(const CcSeqLatentDecode* a, void* stream);
  *   CC_GEMV_PRE_OUTPUT_NORM  s = x + r / sqrt(mean(r^2) + eps) * (w + gain_offset), r = y, or with top > 0 the sum of
  *                            wts[k] * y[k * K ...] over k < top (what cc_seq_post_norm does for one row); s is also
  *                            written to x_out (not x: other CTAs still read it)
- *   CC_GEMV_PRE_GATED_HEADS  y[k] / (root mean square of its part of w_len entries) * w[k mod w_len] * act(gate[k])
+ *   CC_GEMV_PRE_GATED_HEADS  y[k] / (root mean square of its part of part_len entries) * w[k mod w_len] * act(gate[k])
+ *                            (part_len 0 = w_len)
  * conv_rows > 0: rows n < conv_rows of the job then pass a causal convolution over time (a channel per row, the taps
  * before the current one from `tail` fp32 [taps - 1, conv_rows], which is moved on) and the activation conv_act.
+ * post.x set: row n of job 0 is the sublayer's result for channel n and passes cc_seq_bounded_sum's arithmetic on its
+ * way out (post.y, T, E and rows are not used; post.x_out may be post.x; job 0's `out` may then be NULL).
  */
 #define CC_GEMV_MAX_JOBS 6
 #define CC_GEMV_PRE_NONE         0
@@ -283,11 +288,27 @@ typedef struct CcSeqGemvPre {
     int32_t kind, top, w_len, gate_act;
     const float* x;  const float* y;  const float* wts;  const float* w;  const float* gate;  float* x_out;
     float eps, gain_offset;
+    int32_t part_len;
 } CcSeqGemvPre;
+/* See cc_seq_bounded_sum (sixth part). */
+typedef struct CcSeqBounded { const float* alpha;  const float* w;  const float* b; } CcSeqBounded;
+typedef struct CcSeqBoundedSum {
+    const float* x;
+    const float* y;  int64_t ldy;
+    CcSeqBounded out_norm;
+    float mult;
+    const float* add;
+    float* x_out;
+    CcSeqBounded next_norm;
+    void* h;  int32_t act_dtype;
+    const int64_t* rows;
+    int32_t T, E;
+} CcSeqBoundedSum;
 typedef struct CcSeqGemvMulti {
     CcSeqGemvJob job[CC_GEMV_MAX_JOBS];
     int32_t n_jobs, w_dtype;
     CcSeqGemvPre pre;
+    CcSeqBoundedSum post;
 } CcSeqGemvMulti;
 int cc_seq_gemv_multi(const CcSeqGemvMulti* g, void* stream);
 
@@ -462,7 +483,9 @@ int cc_seq_gated_rms_groups(const float* y, const float* gate, int64_t ldg, int3
  * of Dk, v at off_v: G heads of Dv).  q and k heads: divided by their root mean square times q_norm_w / k_norm_w
  * ([Dk], when set), then the first rot_dims entries turned by the angle p * inv_freq[i] for pair i, p = *input_pos + t;
  * v heads: all Dv entries turned by p * v_inv_freq[m] (when set).  Pairs are (2i, 2i + 1) when interleaved, else
- * (i, i + dims / 2).  A pair (a, b) becomes (a cos - b sin, b cos + a sin).  q_out fp32, k_out / v_out in out_dtype.
+ * (i, i + dims / 2).  A pair (a, b) becomes (a cos - b sin, b cos + a sin), times turn_gain for q and k (0 = 1).
+ * q_bias [H * Dk], k_bias [G * Dk], v_bias [G * Dv] (fp32, each optional) are added to the rows first.
+ * q_out fp32, k_out / v_out in out_dtype.
  */
 typedef struct CcSeqQkvRope {
     const float* in;  int64_t ld;
@@ -473,6 +496,8 @@ typedef struct CcSeqQkvRope {
     const int32_t* input_pos;
     float* q_out;  void* k_out;  void* v_out;  int32_t out_dtype;
     int32_t T;
+    const float* q_bias;  const float* k_bias;  const float* v_bias;
+    float turn_gain;
 } CcSeqQkvRope;
 int cc_seq_qkv_rope(const CcSeqQkvRope* a, void* stream);
 
@@ -569,6 +594,51 @@ int cc_seq_post_norm(const CcSeqPostNorm* a, void* stream);
  */
 int cc_seq_post_norm_route(const CcSeqPostNorm* a, const void* Wr, const float* bias, int32_t n, int32_t top, int32_t* ids,
                            float* wts, void* stream);
+
+/* ------------------------------------------------------------------------------------------------------------------
+ * Sixth part (csrc/seq/cell_kernels.cu): element-wise bounded norms around every sublayer, and a matrix memory with
+ * exponential gates.
+ * ------------------------------------------------------------------------------------------------------------------ */
+
+/*
+ * B(v) = w * tanh(*alpha * v) + b, element by element (CcSeqBounded: alpha one fp32 number, w and b fp32 [E]).
+ * Per row t (row rows[t] of x, y and add when `rows` is given; outputs are compact in t):
+ *   s = x[t] + mult * B_out(y[t]) + add[t]           (y and add each optional; fp32, y with row stride ldy)
+ *   x_out[t] = s                                     (optional; may be x itself when rows == NULL)
+ *   h[t] = B_next(s) in act_dtype                    (optional)
+ */
+int cc_seq_bounded_sum(const CcSeqBoundedSum* a, void* stream);
+
+/* x[t] = B_emb(embed[tok[t]]) fp32 [T, E], h[t] = B_next(x[t]) in act_dtype (optional); embed in table_dtype */
+int cc_seq_embed_bounded(const int32_t* tokens, const void* embed, int32_t table_dtype, const CcSeqBounded* emb, float* x,
+                         const CcSeqBounded* next, void* h, int32_t act_dtype, int32_t T, int32_t E, void* stream);
+
+/*
+ * Matrix memory with exponential gates, per head a state S [D, V], a key sum n [D] and a running maximum m.  For each token
+ *   i = cap * tanh((i_raw + i_bias) / cap);   f = logsigmoid(cap * tanh((f_raw + f_bias) / cap))
+ *   m' = max(f + m, i);   S <- exp(f + m - m') S + exp(i - m') k v^T;   n <- the same with k alone;   m <- m'
+ *   o = S^T q / (max(|n . q|, exp(-m)) + den_eps),   q times q_scale
+ * q, k (H * D columns each), v (H * V), i_raw, f_raw (H each): fp32 column ranges with one row stride ld; o fp32
+ * [T, H * V] contiguous; state fp32 [H, D, V] and aux fp32 [H, D + 2] (n, m and a counter
+ * that is zero between calls) are read and written.
+ * path: CC_MLSTM_SCAN runs token by token (D <= 512); CC_MLSTM_CHUNKS in chunks of 64 tokens: state sums of all chunks
+ * at once, a pass over the chunk states, then all chunks' outputs at once (workspace: cc_seq_mlstm_workspace() bytes,
+ * 16-byte aligned); CC_MLSTM_AUTO picks.
+ */
+#define CC_MLSTM_AUTO    0
+#define CC_MLSTM_SCAN    1
+#define CC_MLSTM_CHUNKS  2
+typedef struct CcSeqMlstm {
+    const float* q;  const float* k;  const float* v;  const float* i_raw;  const float* f_raw;  int64_t ld;
+    const float* i_bias;  const float* f_bias;
+    float gate_cap, q_scale, den_eps;
+    float* state;  float* aux;
+    float* o;
+    int32_t T, H, D, V, path;
+    void* workspace;  uint64_t workspace_bytes;
+} CcSeqMlstm;
+uint64_t cc_seq_mlstm_workspace(int32_t T, int32_t H, int32_t D, int32_t V, int32_t path);   /* 0 = none needed */
+int cc_seq_mlstm(const CcSeqMlstm* a, void* stream);
 
 #ifdef __cplusplus
 }
