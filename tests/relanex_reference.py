@@ -123,9 +123,12 @@ MIXERS = {"attention": attention, "latent_attention": latent_attention, "mlstm":
 
 # ------------------------------------------------------------------------------------------------ the model
 
+def silu(z):
+    return z * torch.sigmoid(z)
+
+
 def feed_forward(h, W, p):
-    z = h @ W[p + "gate"].T
-    return (z * torch.sigmoid(z) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+    return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
 def layer_runs(cfg):
