@@ -857,6 +857,46 @@ def _nobodra_model(sz, ff, device, dtype):
     return model.eval()
 
 
+def _relanex_config(sz, extra):
+    """Matrix-memory layers (half as many heads of 128 x 128 as the shape has) alternate with the two attentions: global (the
+    shape's heads, half of each head rotated, frequencies stretched by 4) and windowed latent (the shape's head count and
+    window, 128 key and 128 value columns, the same ranks as the Detatar arm); every layer has the shape's dense
+    feed-forward.  No loop."""
+    E, D = sz["width"], sz["head"]
+    memory = {"heads": sz["heads"] // 2, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    full = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5,
+            "rot": {"base": 500000.0, "dims": D // 2, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}
+    latent = {"heads": sz["heads"], "dim": 128, "vdim": D, "q_rank": extra["q_rank"], "kv_rank": extra["kv_rank"], "scale": 128 ** -0.5,
+              "mask": {"size": sz["window"]}}
+    kinds = ("mlstm", "attention", "mlstm", "latent_attention")
+    mixers = {"mlstm": memory, "attention": full, "latent_attention": latent}
+    layers = [{"type": kinds[i % 4], "mixer": mixers[kinds[i % 4]], "mlp": {"kind": "dense", "ff": sz["ff"]}} for i in range(sz["layers"])]
+    return {"architecture": "Relanex", "vocab": sz["vocab"], "width": E, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": layers}
+
+
+def _relanex_model(sz, extra, device, dtype):
+    from cold_compress_b200.relanex import RelanexTransformer
+    with torch.device(device):
+        model = RelanexTransformer.from_config(_relanex_config(sz, extra), dtype)
+    gen = torch.Generator(device=device).manual_seed(0)
+    with torch.no_grad():
+        for name, p in model.named_parameters():
+            if p.dim() >= 2:
+                p.copy_(torch.empty(p.shape, device=device).normal_(0.0, 0.02, generator=gen))
+            elif name.endswith("alpha"):
+                p.fill_(0.7)
+            elif name.endswith(("weight", "_norm", "norm_w")):
+                p.fill_(1.0)
+            elif name.endswith("f_bias"):
+                p.fill_(3.0)
+        for layer in model.layers:
+            if layer.block.kind == "latent_attention":
+                m = layer.block.mixer
+                H, D, C = m.heads, m.head_dim, m.kv_rank
+                m.w_uk_t.copy_(m.w_ukv[:H * D].reshape(H, D, C).transpose(1, 2))
+    return model.eval()
+
+
 def _llama_model(sz, device):
     from cold_compress_b200.model import ModelArgs, Transformer
     cfg = ModelArgs(block_size=sz["prompt"] + 1024, vocab_size=sz["vocab"], n_layer=sz["layers"], n_head=sz["heads"],
@@ -901,7 +941,7 @@ def run_design(args):
     flush = torch.zeros(64 << 20, dtype=torch.float32, device=device)
     rows = []
     arms = {"detatar": ("detatar", "tidelorn"), "tefovik": ("tefovik", "detatar"),
-            "nevodra": ("nevodra", "detatar"), "nobodra": ("nobodra", "nevodra")}.get(args.design_model, ("tidelorn", "llama"))
+            "nevodra": ("nevodra", "detatar"), "nobodra": ("nobodra", "nevodra"), "relanex": ("relanex", "detatar")}.get(args.design_model, ("tidelorn", "llama"))
     for name in names:
         sz = DESIGN_SIZES[name]
         P = sz["prompt"]
@@ -912,6 +952,7 @@ def run_design(args):
                      _nevodra_model(sz, DETATAR_SIZES[name], device, torch.bfloat16) if arm == "nevodra" else
                      _tefovik_model(sz, device, torch.bfloat16) if arm == "tefovik" else
                      _nobodra_model(sz, NOBODRA_EXPERT_FF[name], device, torch.bfloat16) if arm == "nobodra" else
+                     _relanex_model(sz, DETATAR_SIZES[name], device, torch.bfloat16) if arm == "relanex" else
                      _tidelorn_model(sz, device, torch.bfloat16) if arm == "tidelorn" else _llama_model(sz, device))
             ck = cache_kwargs(dict(slots=1.0, pattern="tile", strategy="full", compressor="recent_global"))
             ck["global_tokens"] = 0
@@ -945,7 +986,7 @@ def run_design(args):
                 torch.cuda.synchronize()
                 dms = a.elapsed_time(b) / args.steps
             wbytes = sum(p.numel() * p.element_size() for n, p in model.named_parameters() if p.dim() >= 2 and "tok_embeddings" not in n and "bigram" not in n)
-            if arm in ("detatar", "nevodra", "nobodra"):      # a token reads `top` experts of each mixture, not all of them, and one copy of W_uk
+            if arm in ("detatar", "nevodra", "nobodra", "relanex"):      # a token reads `top` experts of each mixture, not all of them, and one copy of W_uk
                 for layer in model.layers:
                     block = getattr(layer, "block", layer)
                     f, m = block.mlp, block.mixer
@@ -960,17 +1001,21 @@ def run_design(args):
             del model, decoder
             torch.cuda.empty_cache()
         row["kernels"] = _design_kernels(sz, device, hbm)
-        if args.design_model in ("detatar", "tefovik", "nevodra", "nobodra"):
+        if args.design_model in ("detatar", "tefovik", "nevodra", "nobodra", "relanex"):
             row["detatar_kernels"] = _detatar_kernels(sz, DETATAR_SIZES[name], device, hbm)
         if args.design_model == "nevodra":
             row["nevodra_kernels"] = _nevodra_kernels(sz, DETATAR_SIZES[name], device, hbm)
         if args.design_model == "nobodra":
             row["nevodra_kernels"] = _nevodra_kernels(sz, DETATAR_SIZES[name], device, hbm)
             row["nobodra_kernels"] = _nobodra_kernels(sz, NOBODRA_EXPERT_FF[name], device, hbm)
+        if args.design_model == "relanex":
+            row["relanex_kernels"] = _relanex_kernels(sz, DETATAR_SIZES[name], device, hbm)
+            row["nobodra_kernels"] = _nobodra_kernels(sz, NOBODRA_EXPERT_FF[name], device, hbm)
         if args.design_model in ("tefovik", "nobodra"):
             row["tefovik_kernels"] = _tefovik_kernels(sz, device, hbm)
         rows.append(row)
-    metric = ("prefill and decode tokens/s, Nobodra beside Nevodra at equal layer shape" if args.design_model == "nobodra" else
+    metric = ("prefill and decode tokens/s, Relanex beside Detatar at equal layer shape" if args.design_model == "relanex" else
+              "prefill and decode tokens/s, Nobodra beside Nevodra at equal layer shape" if args.design_model == "nobodra" else
               "prefill and decode tokens/s, Nevodra beside Detatar at equal layer shape" if args.design_model == "nevodra" else
               "prefill and decode tokens/s, Detatar beside Tidelorn at equal layer shape" if args.design_model == "detatar" else
               "prefill and decode tokens/s, Tefovik beside Detatar at equal layer shape" if args.design_model == "tefovik" else
@@ -1304,6 +1349,80 @@ def _nobodra_kernels(sz, ff, device, hbm):
     return out
 
 
+def _relanex_kernels(sz, extra, device, hbm):
+    """The Relanex kernels alone at this shape: the matrix memory over a prompt (in chunks, and by the token scan for
+    comparison) and for one token, the sum between two bounded norms over a prompt, a one-token product with that sum as its
+    way out beside the plain product, and latent attention over a window for a prompt and for one token.  (The global
+    attention is `prefill_attention_global` / `decode_attention_global`.)"""
+    from cold_compress_b200 import _lib, seq_ops
+    from cold_compress_b200.cache import get_cache_constructor
+    cfg = _relanex_config(sz, extra)
+    P, E = sz["prompt"], sz["width"]
+    gen = torch.Generator(device=device).manual_seed(7)
+    out = {}
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=device)
+
+    def token_us(fn, n=20, flush=None):
+        fn(0)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(n):
+                fn(i)
+        return _time_events(graph.replay, 2, 5, flush) * 1e3 / n
+
+    def rate(nbytes, us):
+        return {"us": round(us, 2), "gb_per_s": round(nbytes / us / 1e3, 1), "frac_of_hbm": round(nbytes / us / 1e3 / hbm, 3)}
+
+    m = cfg["layers"][0]["mixer"]
+    H, D, V = m["heads"], m["dim"], m["vdim"]
+    a, b, c, d = H * D, 2 * H * D, 2 * H * D + H * V, 2 * H * D + H * V + H
+    row = torch.randn(P, d + H, device=device, generator=gen)
+    ib, fb = torch.zeros(H, device=device), torch.full((H,), 3.0, device=device)
+    state, aux, o = torch.zeros(H, D, V, device=device), torch.zeros(H, D + 2, device=device), torch.empty(P, H * V, device=device)
+
+    def memory(n, path=_lib.MLSTM_AUTO):
+        r = row[:n]
+        seq_ops.mlstm(r[:, :a], r[:, a:b], r[:, b:c], r[:, c:d], r[:, d:], ib, fb, m["gate_cap"], D ** -0.5, state, aux, o[:n], H, D, V, path=path)
+
+    for label, path in (("memory_prompt", _lib.MLSTM_AUTO), ("memory_prompt_scan", _lib.MLSTM_SCAN)):
+        ms = _time_events(lambda: memory(P, path), 2, 3, flush)
+        # per state entry and token: one update (2) and one read-out (2); the chunk form does other work for the same result
+        out[label] = {"ms": round(ms, 3), "fp32_tflops_of_the_recurrence": round(4.0 * P * H * D * V / ms / 1e9, 2),
+                      "gb_per_s": round((2.0 * H * D + 2 * H * V + 2 * H) * P * 4 / ms / 1e6, 1)}
+    out["memory_token"] = rate(2 * H * D * V * 4, token_us(lambda i: memory(1)))
+    x, y = torch.randn(P, E, device=device, generator=gen), torch.randn(P, E, device=device, generator=gen)
+    norms = [(torch.full((1,), 0.7, device=device), torch.ones(E, device=device), torch.zeros(E, device=device)) for _ in range(2)]
+    h = torch.empty(P, E, device=device, dtype=torch.bfloat16)
+    us = 1e3 * _time_events(lambda: seq_ops.bounded_sum(x, y, norms[0], 0.5, None, x, norms[1], h), 2, 3, flush)
+    out["bounded_sum_prompt"] = rate(P * E * (3 * 4 + 2), us)          # y read, x read and written, bf16 copy written
+    F = sz["ff"]
+    ws = [(torch.randn(E, F, device=device, generator=gen) * 0.02).to(torch.bfloat16) for _ in range(8)]      # more than L2 holds
+    inp, plain = torch.randn(1, F, device=device, generator=gen).to(torch.bfloat16), torch.empty(1, E, device=device)
+    post = seq_ops.bounded_way_out(x[:1], norms[0], 0.5, x[:1], norms[1], h[:1])
+    out["product_token_with_way_out"] = rate(E * F * 2, token_us(lambda i: seq_ops.gemv_multi([(inp, ws[i], None)], post=post), 8, flush))
+    out["product_token_plain"] = rate(E * F * 2, token_us(lambda i: seq_ops.gemv_multi([(inp, ws[i], plain)]), 8, flush))
+    del ws
+    l = cfg["layers"][3]["mixer"]
+    Hq, Dk, Dv, C, W = l["heads"], l["dim"], l["vdim"], l["kv_rank"], l["mask"]["size"]
+    q = torch.randn(P, Hq, Dk, device=device, generator=gen)
+    k, v = torch.randn(P, Hq, Dk, device=device, generator=gen).to(torch.bfloat16), torch.randn(P, Hq, Dv, device=device, generator=gen).to(torch.bfloat16)
+    yy, ip0 = torch.empty(P, Hq, Dv, device=device, dtype=torch.bfloat16), torch.zeros(1, dtype=torch.int32, device=device)
+    ms = _time_events(lambda: seq_ops.attention_rows(q, k, v, None, None, None, ip0, yy, Dk ** -0.5, window=W), 2, 3)
+    pairs = sum(min(i + 1, W) for i in range(P))
+    out["prefill_attention_latent_window"] = {"ms": round(ms, 3), "fp32_tflops": round(2.0 * pairs * (Dk + Dv) * Hq / ms / 1e9, 2)}
+    ctor, _ = get_cache_constructor("latent")
+    with torch.device(device):
+        cache = ctor(1, 1, C, torch.bfloat16, max_cache_length=W, max_seq_length=P + 8, global_tokens=0, cache_bits=None)
+    rows = torch.randn(P, 1, C, device=device, generator=gen).to(torch.bfloat16)
+    cache.sequence_append(rows, ip0)
+    ql, yl = torch.randn(1, Hq, C, device=device, generator=gen), torch.empty(1, Hq, C, device=device, dtype=torch.bfloat16)
+    ipd = torch.tensor([P], dtype=torch.int32, device=device)
+    us = token_us(lambda i: cache.latent_step(ql, rows[:1], ipd, yl, 0.1, window=W))
+    out["decode_attention_latent_window"] = dict(rate(W * C * 2, us), launches=2, fp32_tflops=round(4.0 * W * Hq * C / us / 1e6, 2))
+    return out
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1316,9 +1435,9 @@ def main():
     ap.add_argument("--design", default="", metavar="SIZES",
                     help="instead of the headline workload: Tidelorn beside the Llama-family model at equal layer shape, "
                          "comma-separated sizes of " + "/".join(DESIGN_SIZES))
-    ap.add_argument("--design-model", default="tidelorn", choices=["tidelorn", "detatar", "tefovik", "nevodra", "nobodra"],
+    ap.add_argument("--design-model", default="tidelorn", choices=["tidelorn", "detatar", "tefovik", "nevodra", "nobodra", "relanex"],
                     help="with --design: which design is measured (tidelorn: beside the Llama-family model; detatar: beside "
-                         "Tidelorn; tefovik, nevodra: beside Detatar; nobodra: beside Nevodra; sizes " + "/".join(DETATAR_SIZES) + ")")
+                         "Tidelorn; tefovik, nevodra, relanex: beside Detatar; nobodra: beside Nevodra; sizes " + "/".join(DETATAR_SIZES) + ")")
     args = ap.parse_args()
     if args.design:
         return run_design(args)
