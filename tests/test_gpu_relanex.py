@@ -242,9 +242,9 @@ def test_memory_with_saturated_gates(cap, i_mean, f_mean):
 def test_an_old_write_is_read_back_where_the_gate_kept_it(portions, path):
     """A key that only position 7 writes is asked for at the last position: a head whose forget gate stays open returns its
     value, a head whose gate is half closed has lost it."""
-    if path == 2 and len(portions) > 100:
-        pytest.skip("one-token steps take the scan")
     H, D, V, T = 2, 24, 10, 900
+    if path == 2 and len(portions) > 100:      # single tokens are the scan's
+        portions = (1, 1, 9, 64, 2, T - 77)
     q, k, v, i, f, ib, fb = _memory_inputs(H, D, V, T, 3)
     for h in range(H):
         k[:, h * D] = q[:, h * D] = 0.0
